@@ -3,7 +3,8 @@
 Layers whose mixers ask for the same kind of pages (kv heads, head size,
 window) form a *group*: one page id addresses that page in every layer of the
 group, and each request has one block list per group.  Groups with a window
-give pages back as soon as the window has moved past them; all groups give
+give pages back as soon as the window has moved past them (but for the pages of the first tokens, where a mixer
+keeps seeing those); all groups give
 everything back when a request ends.  Freed pages are handed out again.
 Beside the pages, every live request holds one *state slot*, the row of its
 block tables and of every fixed-size state tensor a mixer declared.
@@ -236,10 +237,11 @@ class CacheManager:
             if w is None:
                 continue
             blocks = rc.blocks[group.index]
+            kept = -(-group.requirement.keep_first // self.block_size)      # pages of the first tokens stay
             # the next token sits at position >= num_tokens and sees keys >= num_tokens - w + 1
             dead = max(0, (rc.num_tokens - w + 1)) // self.block_size
             release = []
-            for b in range(min(dead, len(blocks))):
+            for b in range(kept, min(dead, len(blocks))):
                 if blocks[b] >= 0:
                     release.append(blocks[b])
                     blocks[b] = -1

@@ -11,7 +11,9 @@
 // i.e. attention with ONE key/value head of width rank + rot whose values are the first rank columns of
 // the keys.  Kernels here:
 //   latent_prep       per token: c = rms(down[:rank]) * w, kr = rotate(down[rank:]), both stored into the
-//                     token's cache slot; the rotated part of every query head is rotated in place
+//                     token's cache slot; the rotated part of every query head is rotated in place.  Where the
+//                     queries go through a latent of their own, that latent is RMS-normed here instead and
+//   latent_rotate_q   rotates the query heads made from it
 //   head_linear       out[n, h, :] = W[h] x[n, h, :] for every head (qa from q; values from the summed latents)
 //   attention_latent  softmax attention of every (token, head) over the request's cached [c ; kr], with an
 //                     optional sigmoid gate per (token, head) on the result; CUDA cores, any widths
@@ -35,7 +37,7 @@ latent_prep_kernel(T* __restrict__ rows, int64_t stride, const float* __restrict
                    const int* __restrict__ positions, const float* __restrict__ inv_freq,
                    const int* __restrict__ slot_mapping, T* __restrict__ cache, int n_tokens, int heads, int q_head,
                    int q_plain, int down_col, int rank, int rot, int rot_dims, int block_size, int num_pages,
-                   int* __restrict__ status) {
+                   int q_rank, const float* __restrict__ q_norm_w, T* __restrict__ q_latent, int* __restrict__ status) {
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
@@ -59,6 +61,16 @@ latent_prep_kernel(T* __restrict__ rows, int64_t stride, const float* __restrict
     const float u = to_float(part[2 * i]), v = to_float(part[2 * i + 1]);
     part[2 * i] = from_float<T>(u * c - v * s);
     part[2 * i + 1] = from_float<T>(v * c + u * s);
+  }
+  if (q_rank > 0) {          // the queries' latent: the row's first q_rank columns
+    float qs = 0.f;
+    for (int c = threadIdx.x; c < q_rank; c += blockDim.x) {
+      const float x = to_float(row[c]);
+      qs = fmaf(x, x, qs);
+    }
+    const float q_inv = 1.0f / sqrtf(block_sum(qs, scratch) / (float)q_rank + eps);
+    for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
+      q_latent[(size_t)n * q_rank + c] = from_float<T>(to_float(row[c]) * q_inv * q_norm_w[c]);
   }
   const T* down = row + down_col;
   float ss = 0.f;
@@ -85,6 +97,26 @@ latent_prep_kernel(T* __restrict__ rows, int64_t stride, const float* __restrict
     dst[rank + 2 * i + 1] = from_float<T>(v * c + u * s);
   }
   for (int c = rot_dims + threadIdx.x; c < rot; c += blockDim.x) dst[rank + c] = down[rank + c];
+}
+
+// One thread per (token, head, pair): neighbours (2i, 2i+1) of the rotated part of every query head, in place.
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_rotate_q_kernel(T* __restrict__ rows, int64_t stride, const int* __restrict__ positions,
+                       const float* __restrict__ inv_freq, int n_tokens, int heads, int q_head, int q_plain, int half) {
+  pdl_trigger();
+  pdl_wait();
+  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const int per_token = heads * half;
+  const int64_t n = idx / per_token;
+  if (n >= n_tokens) return;
+  const int u = (int)(idx - n * per_token), h = u / half, i = u - h * half;
+  float s, c;
+  sincosf((float)positions[n] * inv_freq[i], &s, &c);
+  T* part = rows + n * stride + (int64_t)h * q_head + q_plain + 2 * i;
+  const float a = to_float(part[0]), b = to_float(part[1]);
+  part[0] = from_float<T>(a * c - b * s);
+  part[1] = from_float<T>(b * c + a * s);
 }
 
 // ------------------------------------------------------------------ head_linear
@@ -235,15 +267,28 @@ int latent_prep_launch(T* rows, int64_t stride, const float* parts, int n_parts,
                        const float* norm_w, float eps, const int* positions,
                        const float* inv_freq, const int* slot_mapping, T* cache, int n_tokens, int heads, int q_head,
                        int q_plain, int down_col, int rank, int rot, int rot_dims, int block_size, int num_pages,
-                       int* status, cudaStream_t stream) {
+                       int q_rank, const float* q_norm_w, T* q_latent, int* status, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (rank <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || rot_dims % 2 || q_plain + rot > q_head ||
-      n_parts > 16 || (parts && width > stride))
+      n_parts > 16 || (parts && width > stride) ||
+      (q_rank > 0 && (q_norm_w == nullptr || q_latent == nullptr || q_rank > down_col)))
     return (int)cudaErrorInvalidValue;
   return gllm_launch(latent_prep_kernel<T>, dim3((unsigned)n_tokens), dim3(256), 0, stream, rows, stride, parts,
                      n_parts, part_stride, width, norm_w, eps,
                      positions, inv_freq, slot_mapping, cache, n_tokens, heads, q_head, q_plain, down_col, rank, rot,
-                     rot_dims, block_size, num_pages, status);
+                     rot_dims, block_size, num_pages, q_rank, q_norm_w, q_latent, status);
+}
+
+template <typename T>
+int latent_rotate_q_launch(T* rows, int64_t stride, const int* positions, const float* inv_freq, int n_tokens, int heads,
+                           int q_head, int q_plain, int half, cudaStream_t stream) {
+  if (n_tokens <= 0 || half <= 0) return 0;
+  if (heads <= 0 || q_plain < 0 || q_plain + 2 * half > q_head || (int64_t)heads * q_head > stride)
+    return (int)cudaErrorInvalidValue;
+  const int64_t blocks = ((int64_t)n_tokens * heads * half + 255) / 256;
+  if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
+  return gllm_launch(latent_rotate_q_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, rows, stride, positions,
+                     inv_freq, n_tokens, heads, q_head, q_plain, half);
 }
 
 template <typename T>
@@ -285,12 +330,18 @@ int attention_latent_launch(const T* qa, int64_t qa_stride, int qa_head, const T
                                     int width, const float* norm_w, float eps, const int* positions,             \
                                     const float* inv_freq, const int* slot_mapping, T* cache, int n_tokens,      \
                                     int heads, int q_head, int q_plain, int down_col, int rank, int rot,         \
-                                    int rot_dims, int block_size, int num_pages, int* status,                    \
-                                    cudaStream_t stream) {                                                       \
+                                    int rot_dims, int block_size, int num_pages, int q_rank,                     \
+                                    const float* q_norm_w, T* q_latent, int* status, cudaStream_t stream) {      \
     return latent_prep_launch<T>(rows, stride, parts, n_parts, part_stride, width, norm_w, eps, positions,       \
                                  inv_freq, slot_mapping, cache, n_tokens,                                        \
                                  heads, q_head, q_plain, down_col, rank, rot, rot_dims, block_size, num_pages,   \
-                                 status, stream);                                                                \
+                                 q_rank, q_norm_w, q_latent, status, stream);                                    \
+  }                                                                                                              \
+  GLLM_API int gllm_latent_rotate_q_##S(T* rows, int64_t stride, const int* positions, const float* inv_freq,    \
+                                        int n_tokens, int heads, int q_head, int q_plain, int half,              \
+                                        cudaStream_t stream) {                                                   \
+    return latent_rotate_q_launch<T>(rows, stride, positions, inv_freq, n_tokens, heads, q_head, q_plain, half,  \
+                                     stream);                                                                    \
   }                                                                                                              \
   GLLM_API int gllm_head_linear_##S(const T* x, int64_t x_stride, int x_head, const T* w, T* out,                \
                                     int64_t out_stride, int out_head, int n_tokens, int heads, int I, int J,     \

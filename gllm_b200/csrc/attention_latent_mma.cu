@@ -12,7 +12,9 @@
 // Key tiles are aligned to absolute positions, so a token's result does not depend on how its request was cut
 // into steps.  With `splits` > 1 a CTA visits the key tiles [s * tiles_per_split, (s + 1) * tiles_per_split)
 // only and leaves (unnormalised O, maximum, sum) in fp32; latent_merge combines the ranges (single decoded
-// tokens over a long context get enough CTAs that way).  The per-head sigmoid gate multiplies the result.
+// tokens over a long context get enough CTAs that way).  The per-head sigmoid gate multiplies the result.  RANK and
+// ROT are the widths the tiles are built for; the cached vectors may be narrower in either part (multiples of 8): the
+// rest of a tile is zero.  With a window w only keys less than w positions back are visited.
 #include "mma_utils.cuh"
 
 namespace {
@@ -41,8 +43,8 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
                   float* __restrict__ part_ml, const __nv_bfloat16* __restrict__ cache,
                   const int* __restrict__ block_table, int bt_stride, const int* __restrict__ cu_q,
                   const int* __restrict__ ctx_lens, const int* __restrict__ slots, int n_tokens, int heads, int gp,
-                  int qt, int q_rows, int block_size, int num_pages, float scale_log2, int splits,
-                  int tiles_per_split, int* __restrict__ status) {
+                  int qt, int q_rows, int rank, int rot, int block_size, int num_pages, float scale_log2, int window,
+                  int splits, int tiles_per_split, int* __restrict__ status) {
   constexpr int DK = RANK + ROT, CK = DK / 8, CR = RANK / 8, CP = LM_BN / 8;
   constexpr int K_BYTES = LM_BN * DK * 2;
   // q_rows: a multiple of 16 that no CTA of the launch uses more rows than (16 for single tokens of 16 heads: the
@@ -81,9 +83,10 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
   const int rb = (warp & 3) * 16, half = warp >> 2;
 
   const int pos_first = ctx + t0, pos_last = ctx + t0 + t_count - 1;
-  int tile_first = 0, tile_last = pos_last / LM_BN;
+  const int wstart = window > 0 ? max(0, pos_first - window + 1) : 0;      // the first key any row sees
+  int tile_first = wstart / LM_BN, tile_last = pos_last / LM_BN;
   if (splits > 1) {
-    tile_first = split * tiles_per_split;
+    tile_first += split * tiles_per_split;
     tile_last = min(tile_last, tile_first + tiles_per_split - 1);
   }
 
@@ -114,18 +117,21 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
         const int tl = rr / gp, g = rr - tl * gp;
         const bool ok = rr < rows_used;
         const int64_t token = tok_begin + t0 + (ok ? tl : 0);
-        const __nv_bfloat16* a_src = qa + token * qa_stride + (int64_t)(h0 + (ok ? g : 0)) * RANK;
+        const __nv_bfloat16* a_src = qa + token * qa_stride + (int64_t)(h0 + (ok ? g : 0)) * rank;
         const __nv_bfloat16* r_src = qr + token * qr_stride + (int64_t)(h0 + (ok ? g : 0)) * qr_head;
-        for (int piece = threadIdx.x & 3; piece < CK; piece += 4)
+        for (int piece = threadIdx.x & 3; piece < CK; piece += 4) {
+          const bool plain = piece < CR;
+          const bool take = ok && (plain ? piece * 8 < rank : (piece - CR) * 8 < rot);
           cp_async16(smem_u32(q_sm + (rr * CK + lswz<CK>(rr, piece)) * 16),
-                     piece < CR ? a_src + piece * 8 : r_src + (piece - CR) * 8, ok);
+                     take ? (plain ? a_src + piece * 8 : r_src + (piece - CR) * 8) : qa, take);
+        }
       }
     }
     auto load_k = [&](int tile, int stage) {     // eight threads a key: one look-up of its page per thread
       unsigned char* dst = k_sm0 + stage * K_BYTES;
       const int row = threadIdx.x >> 3;
       const int key = tile * LM_BN + row;
-      bool ok = key <= pos_last;
+      bool ok = key <= pos_last && key >= wstart;       // (a page before the window may have been given back)
       int page = 0;
       if (ok) {
         page = bt[key / block_size];
@@ -135,9 +141,13 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
           page = 0;
         }
       }
-      const __nv_bfloat16* src = ok ? cache + ((int64_t)page * block_size + key % block_size) * DK : cache;
-      for (int piece = threadIdx.x & 7; piece < CK; piece += 8)
-        cp_async16(smem_u32(dst + (row * CK + lswz<CK>(row, piece)) * 16), ok ? src + piece * 8 : cache, ok);
+      const __nv_bfloat16* src = ok ? cache + ((int64_t)page * block_size + key % block_size) * (rank + rot) : cache;
+      for (int piece = threadIdx.x & 7; piece < CK; piece += 8) {
+        const bool plain = piece < CR;
+        const bool take = ok && (plain ? piece * 8 < rank : (piece - CR) * 8 < rot);
+        cp_async16(smem_u32(dst + (row * CK + lswz<CK>(row, piece)) * 16),
+                   take ? src + (plain ? piece * 8 : rank + (piece - CR) * 8) : cache, take);
+      }
     };
     load_k(tile_first, 0);
     cp_async_commit();
@@ -221,7 +231,7 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
           float x = s_sm[srow * S_LD + squart * 8 + e];
           if (FEW) x += s_sm[(16 + srow) * S_LD + squart * 8 + e];      // the other half of the width
           x *= scale_log2;
-          v[e] = (s_ok && key <= s_qpos) ? x : -INFINITY;
+          v[e] = (s_ok && key <= s_qpos && (window <= 0 || s_qpos - key < window)) ? x : -INFINITY;
           mx = fmaxf(mx, v[e]);
         }
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -330,11 +340,12 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
           const int col = pair * 16 + nt * 8 + 2 * t4;
+          if (col >= rank) continue;
           if (splits > 1)
-            *reinterpret_cast<float2*>(part_o + (((int64_t)split * n_tokens + token) * heads + head) * RANK + col) =
+            *reinterpret_cast<float2*>(part_o + (((int64_t)split * n_tokens + token) * heads + head) * rank + col) =
                 make_float2(of[j][nt][2 * i], of[j][nt][2 * i + 1]);
           else
-            *reinterpret_cast<__nv_bfloat162*>(out + token * out_stride + (int64_t)head * RANK + col) =
+            *reinterpret_cast<__nv_bfloat162*>(out + token * out_stride + (int64_t)head * rank + col) =
                 __floats2bfloat162_rn(of[j][nt][2 * i] * mult, of[j][nt][2 * i + 1] * mult);
         }
       }
@@ -349,10 +360,10 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
     const int head = h0 + g;
     const int col0 = half * (RANK / 2);
     if (splits > 1) {
-      float* dst = part_o + (((int64_t)split * n_tokens + token) * heads + head) * RANK + col0;
+      float* dst = part_o + (((int64_t)split * n_tokens + token) * heads + head) * rank + col0;
 #pragma unroll
       for (int nd = 0; nd < NV; ++nd)
-        *reinterpret_cast<float2*>(dst + nd * 8 + 2 * t4) = make_float2(o[nd][2 * i], o[nd][2 * i + 1]);
+        if (col0 + nd * 8 < rank) *reinterpret_cast<float2*>(dst + nd * 8 + 2 * t4) = make_float2(o[nd][2 * i], o[nd][2 * i + 1]);
       if (half == 0 && t4 == 0) {
         float* ml = part_ml + (((int64_t)split * n_tokens + token) * heads + head) * 2;
         ml[0] = m_sm[rr];
@@ -362,10 +373,10 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ qa, int64_t qa_stride, const
       const float l = l_sm[rr];
       float mult = l > 0.f ? 1.0f / l : 0.f;
       if (gate) mult *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[token * gate_stride + head])));
-      __nv_bfloat16* dst = out + token * out_stride + (int64_t)head * RANK + col0;
+      __nv_bfloat16* dst = out + token * out_stride + (int64_t)head * rank + col0;
 #pragma unroll
       for (int nd = 0; nd < NV; ++nd)
-        *reinterpret_cast<__nv_bfloat162*>(dst + nd * 8 + 2 * t4) =
+        if (col0 + nd * 8 < rank) *reinterpret_cast<__nv_bfloat162*>(dst + nd * 8 + 2 * t4) =
             __floats2bfloat162_rn(o[nd][2 * i] * mult, o[nd][2 * i + 1] * mult);
     }
   }
@@ -514,8 +525,8 @@ int latent_mma_launch(const __nv_bfloat16* qa, int64_t qa_stride, const __nv_bfl
                       int qr_head, const __nv_bfloat16* gate, int64_t gate_stride, __nv_bfloat16* out,
                       int64_t out_stride, float* part_o, float* part_ml, const __nv_bfloat16* cache,
                       const int* block_table, int bt_stride, const int* cu_q, const int* ctx_lens, const int* slots,
-                      int num_requests, int max_q_len, int n_tokens, int heads, int block_size, int num_pages,
-                      float scale, int splits, int tiles_per_split, int* status, cudaStream_t stream) {
+                      int num_requests, int max_q_len, int n_tokens, int heads, int rank, int rot, int block_size,
+                      int num_pages, float scale, int window, int splits, int tiles_per_split, int* status, cudaStream_t stream) {
   const int gp = heads <= LM_BM ? heads : 1;
   const int qt = LM_BM / gp;
   const int rows_most = (max_q_len < qt ? max_q_len : qt) * gp;
@@ -536,19 +547,20 @@ int latent_mma_launch(const __nv_bfloat16* qa, int64_t qa_stride, const __nv_bfl
   auto kernel = q_rows == 16 ? latent_mma_kernel<RANK, ROT, true> : latent_mma_kernel<RANK, ROT, false>;
   int code = gllm_launch(kernel, grid, dim3(LM_THREADS), smem, stream, qa, qa_stride, qr,
                          qr_stride, qr_head, gate, gate_stride, out, out_stride, part_o, part_ml, cache, block_table,
-                         bt_stride, cu_q, ctx_lens, slots, n_tokens, heads, gp, qt, q_rows, block_size, num_pages,
-                         scale * LOG2E, splits, tiles_per_split, status);
+                         bt_stride, cu_q, ctx_lens, slots, n_tokens, heads, gp, qt, q_rows, rank, rot, block_size,
+                         num_pages, scale * LOG2E, window, splits, tiles_per_split, status);
   if (code != 0 || splits <= 1) return code;
   return gllm_launch(latent_merge_kernel, dim3((unsigned)(n_tokens * heads)), dim3(RANK >= 512 ? 512 : 256), 0, stream,
                      (const float*)part_o, (const float*)part_ml, gate, gate_stride, out, out_stride, n_tokens, heads,
-                     RANK, splits);
+                     rank, splits);
 }
 }  // namespace
 
+// narrowest first: a launch takes the first one that holds both widths
 #define GLLM_LATENT_SIZES(X) X(64, 32) X(64, 64) X(96, 32) X(128, 32) X(128, 64) X(256, 32) X(256, 64) X(512, 64)
 
 GLLM_API int gllm_attention_latent_mma_supports(int rank, int rot) {
-#define GLLM_LM_OK(A, B) if (rank == A && rot == B) return 1;
+#define GLLM_LM_OK(A, B) if (rank > 0 && rot >= 0 && rank % 8 == 0 && rot % 8 == 0 && rank <= A && rot <= B) return 1;
   GLLM_LATENT_SIZES(GLLM_LM_OK)
 #undef GLLM_LM_OK
   return 0;
@@ -563,18 +575,18 @@ GLLM_API int gllm_attention_latent_mma(const __nv_bfloat16* qa, int64_t qa_strid
                                        float* part_ml, const __nv_bfloat16* cache, const int* block_table,
                                        int bt_stride, const int* cu_q, const int* ctx_lens, const int* slots,
                                        int num_requests, int max_q_len, int n_tokens, int heads, int rank, int rot,
-                                       int block_size, int num_pages, float scale, int splits, int tiles_per_split,
-                                       int* status, cudaStream_t stream) {
+                                       int block_size, int num_pages, float scale, int window, int splits,
+                                       int tiles_per_split, int* status, cudaStream_t stream) {
   if (num_requests <= 0 || max_q_len <= 0) return 0;
   if (heads <= 0 || num_requests > 65535 || (qa_stride % 8) || (qr_stride % 8) || (qr_head % 8) || (out_stride % 2) ||
-      splits < 1 || splits > 64 || (splits > 1 && (part_o == nullptr || part_ml == nullptr || tiles_per_split < 1)))
+      rank <= 0 || rot < 0 || (rank % 8) || (rot % 8) || window < 0 || splits < 1 || splits > 64 || (splits > 1 && (part_o == nullptr || part_ml == nullptr || tiles_per_split < 1)))
     return (int)cudaErrorInvalidValue;
 #define GLLM_LM(A, B)                                                                                              \
-  if (rank == A && rot == B)                                                                                       \
+  if (rank <= A && rot <= B)                                                                                       \
     return latent_mma_launch<A, B>(qa, qa_stride, qr, qr_stride, qr_head, gate, gate_stride, out, out_stride,      \
                                    part_o, part_ml, cache, block_table, bt_stride, cu_q, ctx_lens, slots,          \
-                                   num_requests, max_q_len, n_tokens, heads, block_size, num_pages, scale, splits, \
-                                   tiles_per_split, status, stream);
+                                   num_requests, max_q_len, n_tokens, heads, rank, rot, block_size, num_pages,     \
+                                   scale, window, splits, tiles_per_split, status, stream);
   GLLM_LATENT_SIZES(GLLM_LM)
 #undef GLLM_LM
   return (int)cudaErrorInvalidValue;

@@ -12,6 +12,7 @@
 // and add their parts of the two dot products by shuffles.  o_c is formed as (g s).q + u_c (k.q), which needs
 // one round of shuffles per token instead of two.  The state is stored column by column, [slots, heads, dv, dk],
 // as the other matrix recurrences store theirs.
+// The decays come per key channel, g [n, heads * dk], or one per head, g [n, heads] (`decay_width` dk or 1).
 // The flat batch holds prompt portions beside single tokens: request r owns rows cu_q[r] .. cu_q[r+1]-1 and row
 // state_slots[r] of the state tensors, so a prompt may be cut anywhere.
 #include "common.cuh"
@@ -24,7 +25,8 @@ __device__ __forceinline__ float softplusf_(float x) { return fmaxf(x, 0.f) + lo
 constexpr int DELTA_MAX_TAPS = 16;
 
 // x [n, >= channels] at x_stride: the projections' output, q | k | v channels first (qk_cols = 2 * kv_heads * dk,
-// then heads * dv).  Outputs fp32: qk [n, qk_cols], v [n, heads * dv], g [n, heads * dk], beta [n, heads].
+// then heads * dv).  Outputs fp32: qk [n, qk_cols], v [n, heads * dv], g [n, heads * decay_width] (a_raw
+// and dt_bias alike), beta [n, heads].
 // The work of a token is cut into units, one warp each: a q or k head (convolution, SiLU, unit norm: dk channels),
 // or a v head (dv channels) together with that head's decays and beta.  grid.y blocks share a token's units, so a
 // step of few tokens still fills the SMs.  `single` says that every request brings exactly one token: the thread
@@ -38,7 +40,7 @@ delta_prep_kernel(const T* __restrict__ x, int64_t x_stride, const float* __rest
                   const float* __restrict__ dt_bias, const float* __restrict__ A_log,
                   const float* __restrict__ b_raw, int64_t b_stride, float* __restrict__ qk, float* __restrict__ v,
                   float* __restrict__ g, float* __restrict__ beta, int heads, int kv_heads, int dk, int dv, int taps,
-                  float unit_eps, float q_scale, int single) {
+                  float unit_eps, float q_scale, int single, int decay_width) {
   extern __shared__ float sm[];
   pdl_trigger();
   pdl_wait();
@@ -90,9 +92,9 @@ delta_prep_kernel(const T* __restrict__ x, int64_t x_stride, const float* __rest
       for (int c = lane; c < dk; c += 32) qk[(int64_t)i * qk_cols + c0 + c] = mine[c] * inv;
     } else {
       const float rate = -expf(A_log[h]);
-      for (int c = lane; c < dk; c += 32) {
-        const int hc = h * dk + c;
-        g[(int64_t)i * heads * dk + hc] = expf(rate * softplusf_(a_raw[(int64_t)i * a_stride + hc] + dt_bias[hc]));
+      for (int c = lane; c < decay_width; c += 32) {
+        const int hc = h * decay_width + c;
+        g[(int64_t)i * heads * decay_width + hc] = expf(rate * softplusf_(a_raw[(int64_t)i * a_stride + hc] + dt_bias[hc]));
       }
       if (lane == 0) beta[(int64_t)i * heads + h] = sigmoidf_(b_raw[(int64_t)i * b_stride + h]);
     }
@@ -133,12 +135,13 @@ template <int N> __device__ __forceinline__ void copy_async_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
-// Tokens are taken in chunks of `tc`, in two buffers: q [tc][dkp], k [tc][dkp], g [tc][dkp], v [tc][cols], beta [tc]
+// Tokens are taken in chunks of `tc`, in two buffers: q [tc][dkp], k [tc][dkp], g [tc][dkp] (HEAD: [tc], one decay per
+// head), v [tc][cols], beta [tc]
 // (dkp = lanes * DPT >= dk; what lies beyond dk or dv is zeroed once and never copied over).  VEC = 4 copies and
 // reads four floats at a time, which needs dk and dv to be multiples of 4 (all row starts are then 16-byte aligned).
 // Per token the chain from state to state is: dot products with the decayed key and query (the decay is folded
 // into them, off the chain), their sums over the column's lanes, u, one fused multiply-add per state element.
-template <int DPT, int LANES, int VEC>
+template <int DPT, int LANES, int VEC, bool HEAD>
 __global__ void __launch_bounds__(DELTA_THREADS)
 delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float* __restrict__ g,
                   const float* __restrict__ beta, float* __restrict__ state, const int* __restrict__ cu_q,
@@ -154,7 +157,10 @@ delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
   const bool live = col < dv;
   const int t0 = cu_q[r], t1 = cu_q[r + 1];
   if (t1 <= t0) return;
-  const int buf_floats = (tc * (3 * dkp + cols + 1) + 3) & ~3;
+  constexpr int gw = HEAD ? 1 : dkp;                       // decays of a token in shared memory
+  // (a token's decay per head lies behind its beta)
+  const int buf_floats = (tc * (2 * dkp + gw + cols + 1) + 3) & ~3;
+  const int gs_at = HEAD ? tc * (2 * dkp + cols + 1) : 2 * tc * dkp, vs_at = tc * (2 * dkp + (HEAD ? 0 : dkp));
   for (int i = threadIdx.x; i < 2 * buf_floats; i += DELTA_THREADS) sm[i] = 0.f;
   float S[DPT];
   float* sp = state + (((int64_t)state_slots[r] * heads + h) * dv + (live ? col : 0)) * dk + sub * DPT;
@@ -172,26 +178,29 @@ delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
   const int dkv = dk / VEC, colv = cols / VEC;            // cols is a power of two >= 4
   const float* q_src = qk + hg * dk;
   const float* k_src = qk + (kv_heads + hg) * dk;
-  const float* g_src = g + (int64_t)h * dk;
+  const float* g_src = HEAD ? g + h : g + (int64_t)h * dk;
   const float* v_src = v + (int64_t)h * dv + col0;
   auto issue = [&](int c0, int nt, float* buf) {
     float* qs = buf;
     float* ks = qs + tc * dkp;
-    float* gs = ks + tc * dkp;
-    float* vs = gs + tc * dkp;
+    float* gs = buf + gs_at;
+    float* vs = buf + vs_at;
     float* bs = vs + tc * cols;
     for (int idx = threadIdx.x; idx < nt * dkv; idx += DELTA_THREADS) {
       const int t = idx / dkv, d = (idx - t * dkv) * VEC;
       const int64_t tok = c0 + t;
       copy_async(qs + t * dkp + d, q_src + tok * qk_cols + d, VEC);
       copy_async(ks + t * dkp + d, k_src + tok * qk_cols + d, VEC);
-      copy_async(gs + t * dkp + d, g_src + tok * heads * dk + d, VEC);
+      if (!HEAD) copy_async(gs + t * dkp + d, g_src + tok * heads * dk + d, VEC);
     }
     for (int idx = threadIdx.x; idx < nt * colv; idx += DELTA_THREADS) {
       const int t = idx / colv, c = (idx - t * colv) * VEC;
       if (col0 + c < dv) copy_async(vs + t * cols + c, v_src + (int64_t)(c0 + t) * heads * dv + c, VEC);
     }
-    for (int t = threadIdx.x; t < nt; t += DELTA_THREADS) copy_async(bs + t, beta + (int64_t)(c0 + t) * heads + h, 1);
+    for (int t = threadIdx.x; t < nt; t += DELTA_THREADS) {
+      copy_async(bs + t, beta + (int64_t)(c0 + t) * heads + h, 1);
+      if (HEAD) copy_async(gs + t, g_src + (int64_t)(c0 + t) * heads, 1);
+    }
     copy_async_commit();
   };
   __syncthreads();                                         // the zeros are there before the first copy lands
@@ -209,29 +218,36 @@ delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
     const float* buf = sm + which * buf_floats;
     const float* qs = buf + sub * DPT;
     const float* ks = qs + tc * dkp;
-    const float* gs = ks + tc * dkp;
-    const float* vs = buf + 3 * tc * dkp + cix;
-    const float* bs = buf + 3 * tc * dkp + tc * cols;
+    const float* gs = buf + gs_at + (HEAD ? 0 : sub * DPT);
+    const float* vs = buf + vs_at + cix;
+    const float* bs = buf + vs_at + tc * cols;
     float* op = out + ((int64_t)c0 * heads + h) * dv + col;
     // What a token brings (k, g, q, k.q summed over the lanes, v, beta) does not depend on the state and is fetched
     // one token ahead, so that the chain from state to state is the decay, two dot products (in ACC partial sums
     // each), their sums over the lanes, u and one fused multiply-add per element.
     constexpr int ACC = DPT >= 16 ? 4 : (DPT >= 8 ? 2 : 1);
-    auto fetch = [&](int t, float (&k_)[DPT], float (&g_)[DPT], float (&q_)[DPT], float& kq_, float& v_, float& b_) {
+    constexpr int GN = HEAD ? 1 : DPT;
+    auto fetch = [&](int t, float (&k_)[DPT], float (&g_)[GN], float (&q_)[DPT], float& kq_, float& v_, float& b_) {
       if (VEC == 4) {
 #pragma unroll
         for (int e = 0; e < DPT; e += 4) {
           const float4 a = *reinterpret_cast<const float4*>(ks + t * dkp + e);
-          const float4 b = *reinterpret_cast<const float4*>(gs + t * dkp + e);
           const float4 c = *reinterpret_cast<const float4*>(qs + t * dkp + e);
           k_[e] = a.x, k_[e + 1] = a.y, k_[e + 2] = a.z, k_[e + 3] = a.w;
-          g_[e] = b.x, g_[e + 1] = b.y, g_[e + 2] = b.z, g_[e + 3] = b.w;
+          if constexpr (!HEAD) {
+            const float4 b = *reinterpret_cast<const float4*>(gs + t * dkp + e);
+            g_[e] = b.x, g_[e + 1] = b.y, g_[e + 2] = b.z, g_[e + 3] = b.w;
+          }
           q_[e] = c.x, q_[e + 1] = c.y, q_[e + 2] = c.z, q_[e + 3] = c.w;
         }
       } else {
 #pragma unroll
-        for (int e = 0; e < DPT; ++e) k_[e] = ks[t * dkp + e], g_[e] = gs[t * dkp + e], q_[e] = qs[t * dkp + e];
+        for (int e = 0; e < DPT; ++e) {
+          k_[e] = ks[t * dkp + e], q_[e] = qs[t * dkp + e];
+          if constexpr (!HEAD) g_[e] = gs[t * dkp + e];
+        }
       }
+      if constexpr (HEAD) g_[0] = gs[t];
       v_ = vs[t * cols];
       b_ = bs[t];
       float part[ACC] = {};
@@ -245,16 +261,16 @@ delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
 #pragma unroll
       for (int o = LANES >> 1; o > 0; o >>= 1) kq_ += __shfl_xor_sync(0xffffffffu, kq_, o);
     };
-    float kk[DPT], gg[DPT], qq[DPT], kq, vv, bb;
+    float kk[DPT], gg[GN], qq[DPT], kq, vv, bb;
     fetch(0, kk, gg, qq, kq, vv, bb);
 #pragma unroll 2
     for (int t = 0; t < nt; ++t) {
-      float nk[DPT], ng[DPT], nq[DPT], nkq, nv, nb;
+      float nk[DPT], ng[GN], nq[DPT], nkq, nv, nb;
       fetch(min(t + 1, nt - 1), nk, ng, nq, nkq, nv, nb);
       float pk[ACC] = {}, pq[ACC] = {};
 #pragma unroll
       for (int e = 0; e < DPT; ++e) {
-        S[e] *= gg[e];
+        S[e] *= gg[HEAD ? 0 : e];
         pk[e % ACC] = fmaf(S[e], kk[e], pk[e % ACC]);
         pq[e % ACC] = fmaf(S[e], qq[e], pq[e % ACC]);
       }
@@ -273,7 +289,9 @@ delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
       for (int e = 0; e < DPT; ++e) S[e] = fmaf(kk[e], u, S[e]);
       if (sub == 0 && live) op[(int64_t)t * heads * dv] = fmaf(u, kq, sq);
 #pragma unroll
-      for (int e = 0; e < DPT; ++e) kk[e] = nk[e], gg[e] = ng[e], qq[e] = nq[e];
+      for (int e = 0; e < DPT; ++e) kk[e] = nk[e], qq[e] = nq[e];
+#pragma unroll
+      for (int e = 0; e < GN; ++e) gg[e] = ng[e];
       kq = nkq, vv = nv, bb = nb;
     }
     __syncthreads();                                       // the next copies go into the buffer just read
@@ -302,11 +320,12 @@ int delta_prep_launch(const T* x, int64_t x_stride, const float* conv_w, float* 
                       const int* token_row, const int* cu_q, const int* state_slots, int num_requests,
                       const float* a_raw, int64_t a_stride, const float* dt_bias, const float* A_log, const float* b_raw,
                       int64_t b_stride, float* qk, float* v, float* g, float* beta, int n_tokens, int heads, int kv_heads,
-                      int dk, int dv, int taps, float unit_eps, float q_scale, int max_q_len, cudaStream_t stream) {
+                      int dk, int dv, int taps, float unit_eps, float q_scale, int max_q_len, int decay_width,
+                      cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   const int channels = 2 * kv_heads * dk + heads * dv, units = 2 * kv_heads + heads, nwarps = 8;
   const size_t smem = sizeof(float) * (size_t)nwarps * dk;
-  if (taps < 1 || taps > DELTA_MAX_TAPS || heads % kv_heads || smem > 48 * 1024 || num_requests > 65535)
+  if (taps < 1 || taps > DELTA_MAX_TAPS || (decay_width != 1 && decay_width != dk) || heads % kv_heads || smem > 48 * 1024 || num_requests > 65535)
     return (int)cudaErrorInvalidValue;
   // a token's units spread over as many blocks as it takes to give every SM a few, at most one unit a warp
   int parts = (4 * 148 + n_tokens - 1) / n_tokens;
@@ -314,7 +333,7 @@ int delta_prep_launch(const T* x, int64_t x_stride, const float* conv_w, float* 
   const int single = max_q_len == 1 && n_tokens == num_requests;
   int rc = gllm_launch(delta_prep_kernel<T>, dim3(n_tokens, parts), dim3(32 * nwarps), smem, stream, x, x_stride, conv_w,
                        conv_state, positions, token_row, a_raw, a_stride, dt_bias, A_log, b_raw, b_stride,
-                       qk, v, g, beta, heads, kv_heads, dk, dv, taps, unit_eps, q_scale, single);
+                       qk, v, g, beta, heads, kv_heads, dk, dv, taps, unit_eps, q_scale, single, decay_width);
   if (rc != 0 || taps == 1 || num_requests <= 0 || single) return rc;
   return gllm_launch(conv_state_update_kernel<T>, dim3((channels + 255) / 256, num_requests), dim3(256), 0, stream, x,
                      x_stride, conv_state, cu_q, state_slots, channels, taps);
@@ -322,9 +341,9 @@ int delta_prep_launch(const T* x, int64_t x_stride, const float* conv_w, float* 
 
 int delta_rule_launch(const float* qk, const float* v, const float* g, const float* beta, float* state,
                       const int* cu_q, const int* state_slots, float* out, int num_requests, int heads, int kv_heads,
-                      int dk, int dv, int max_q_len, cudaStream_t stream) {
+                      int dk, int dv, int max_q_len, int decay_width, cudaStream_t stream) {
   if (num_requests <= 0) return 0;
-  if (heads > 65535 || num_requests > 65535 || dk < 1 || dv < 1 || dk > 512 || heads % kv_heads)
+  if ((decay_width != 1 && decay_width != dk) || heads > 65535 || num_requests > 65535 || dk < 1 || dv < 1 || dk > 512 || heads % kv_heads)
     return (int)cudaErrorInvalidValue;
   // Key channels a thread keeps (DPT).  More of them mean fewer threads a column, so fewer rounds of shuffles and more
   // independent work per warp, but fewer warps in all.  Measured: four for heads of up to 64 key channels and eight
@@ -348,15 +367,20 @@ int delta_rule_launch(const float* qk, const float* v, const float* g, const flo
   const int lanes = pow2_at_least((dk + dpt - 1) / dpt);
   const int cols = DELTA_THREADS / lanes, dkp = lanes * dpt;
   int tc = DELTA_MAX_CHUNK;
-  while (tc > 2 && 2 * tc * (3 * dkp + cols + 1) * sizeof(float) > 96 * 1024) tc >>= 1;
-  const size_t smem = sizeof(float) * 2 * (size_t)((tc * (3 * dkp + cols + 1) + 3) & ~3);
+  const bool head = decay_width == 1 && dk > 1;
+  const int per_token = 2 * dkp + (head ? 1 : dkp) + cols + 1;
+  while (tc > 2 && 2 * tc * per_token * sizeof(float) > 96 * 1024) tc >>= 1;
+  const size_t smem = sizeof(float) * 2 * (size_t)((tc * per_token + 3) & ~3);
   using Kernel = void (*)(const float*, const float*, const float*, const float*, float*, const int*, const int*, float*,
                           int, int, int, int, int);
   Kernel kernel = nullptr;
 #define GLLM_DELTA_PICK(D, L) \
-  if (dpt == D && lanes == L) kernel = vec ? delta_rule_kernel<D, L, 4> : delta_rule_kernel<D, L, 1>;
+  if (dpt == D && lanes == L)                                                           \
+    kernel = head ? (vec ? delta_rule_kernel<D, L, 4, true> : delta_rule_kernel<D, L, 1, true>)            \
+                  : (vec ? delta_rule_kernel<D, L, 4, false> : delta_rule_kernel<D, L, 1, false>);
 #define GLLM_DELTA_PICK4(D, L) \
-  if (dpt == D && lanes == L && vec) kernel = delta_rule_kernel<D, L, 4>;
+  if (dpt == D && lanes == L && vec)                                                    \
+    kernel = head ? delta_rule_kernel<D, L, 4, true> : delta_rule_kernel<D, L, 4, false>;
   GLLM_DELTA_PICK(4, 1) GLLM_DELTA_PICK(4, 2) GLLM_DELTA_PICK(4, 4) GLLM_DELTA_PICK(4, 8) GLLM_DELTA_PICK(4, 16)
   GLLM_DELTA_PICK(4, 32) GLLM_DELTA_PICK(8, 32) GLLM_DELTA_PICK(16, 32)
   GLLM_DELTA_PICK4(8, 1) GLLM_DELTA_PICK4(8, 2) GLLM_DELTA_PICK4(8, 4) GLLM_DELTA_PICK4(8, 8) GLLM_DELTA_PICK4(8, 16)
@@ -395,17 +419,17 @@ int delta_rule_launch(const float* qk, const float* v, const float* g, const flo
                                    const float* dt_bias, const float* A_log, const float* b_raw, int64_t b_stride,     \
                                    float* qk, float* v, float* g, float* beta, int n_tokens, int heads, int kv_heads,  \
                                    int dk, int dv, int taps, float unit_eps, float q_scale, int max_q_len,             \
-                                   cudaStream_t stream) {                                                              \
+                                   int decay_width, cudaStream_t stream) {                                                              \
     return delta_prep_launch<T>(x, x_stride, conv_w, conv_state, positions, token_row, cu_q, state_slots,              \
                                 num_requests, a_raw, a_stride, dt_bias, A_log, b_raw, b_stride, qk, v, g, beta,        \
-                                n_tokens, heads, kv_heads, dk, dv, taps, unit_eps, q_scale, max_q_len, stream);        \
+                                n_tokens, heads, kv_heads, dk, dv, taps, unit_eps, q_scale, max_q_len, decay_width, stream);        \
   }
 GLLM_DELTA_EXPORTS(float, f32)
 GLLM_DELTA_EXPORTS(__nv_bfloat16, bf16)
 
 GLLM_API int gllm_delta_rule(const float* qk, const float* v, const float* g, const float* beta, float* state,
                              const int* cu_q, const int* state_slots, float* out, int num_requests, int heads,
-                             int kv_heads, int dk, int dv, int max_q_len, cudaStream_t stream) {
+                             int kv_heads, int dk, int dv, int max_q_len, int decay_width, cudaStream_t stream) {
   return delta_rule_launch(qk, v, g, beta, state, cu_q, state_slots, out, num_requests, heads, kv_heads, dk, dv, max_q_len,
-                           stream);
+                           decay_width, stream);
 }

@@ -697,12 +697,12 @@ matrix_recurrence_step_kernel(int mode, const T* __restrict__ q, int64_t q_strid
 // --------------------------------------------------------------- per-head output norm
 // One warp per (token, head): o [dv] (fp32, optionally divided by max(|o[dv]|, o[dv+1]) + den_eps, the
 // two extra columns the recurrence wrote), divided by its root mean square, times a weight (shared by
-// the heads when w_head_stride is 0), times sigmoid(gate) when a gate is given.
+// the heads when w_head_stride is 0), times sigmoid(gate), or silu(gate), when a gate is given.
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_kernel(const float* __restrict__ o, int64_t o_stride, int o_cols, int with_den, float den_eps,
                  const float* __restrict__ w, int w_head_stride, const T* __restrict__ gate, int64_t gate_stride,
-                 T* __restrict__ out, int64_t out_stride, int n_tokens, int heads, int dv, float eps) {
+                 int gate_silu, T* __restrict__ out, int64_t out_stride, int n_tokens, int heads, int dv, float eps) {
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -721,7 +721,10 @@ head_norm_kernel(const float* __restrict__ o, int64_t o_stride, int o_cols, int 
   const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
   for (int c = lane; c < dv; c += 32) {
     float x = (with_den ? row[c] * inv_den : row[c]) * inv * w[(int64_t)h * w_head_stride + c];
-    if (gate) x *= sigmoidf_(to_float(gate[(int64_t)t * gate_stride + (int64_t)h * dv + c]));
+    if (gate) {
+      const float z = to_float(gate[(int64_t)t * gate_stride + (int64_t)h * dv + c]);
+      x *= gate_silu ? siluf_(z) : sigmoidf_(z);
+    }
     out[(int64_t)t * out_stride + (int64_t)h * dv + c] = from_float<T>(x);
   }
 }
@@ -898,13 +901,13 @@ int matrix_recurrence_launch(int mode, const T* q, int64_t q_stride, const T* k,
 
 template <typename T>
 int head_norm_launch(const float* o, int64_t o_stride, int o_cols, int with_den, float den_eps, const float* w,
-                     int w_head_stride, const T* gate, int64_t gate_stride, T* out, int64_t out_stride, int n_tokens,
-                     int heads, int dv, float eps, cudaStream_t stream) {
+                     int w_head_stride, const T* gate, int64_t gate_stride, int gate_silu, T* out, int64_t out_stride,
+                     int n_tokens, int heads, int dv, float eps, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   const int64_t blocks = ((int64_t)n_tokens * heads + 3) / 4;
   if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
   return gllm_launch(head_norm_kernel<T>, dim3((unsigned)blocks), dim3(128), 0, stream, o, o_stride, o_cols, with_den,
-                     den_eps, w, w_head_stride, gate, gate_stride, out, out_stride, n_tokens, heads, dv, eps);
+                     den_eps, w, w_head_stride, gate, gate_stride, gate_silu, out, out_stride, n_tokens, heads, dv, eps);
 }
 
 template <typename T>
@@ -961,11 +964,11 @@ int conv_state_advance_launch(const T* x, int64_t x_stride, float* conv_state, c
                                        num_requests, max_q_len, heads, dk, dv, kv_div, stream);                       \
   }                                                                                                                   \
   GLLM_API int gllm_head_norm_##S(const float* o, int64_t o_stride, int o_cols, int with_den, float den_eps,          \
-                                  const float* w, int w_head_stride, const T* gate, int64_t gate_stride, T* out,      \
-                                  int64_t out_stride, int n_tokens, int heads, int dv, float eps,                     \
-                                  cudaStream_t stream) {                                                              \
-    return head_norm_launch<T>(o, o_stride, o_cols, with_den, den_eps, w, w_head_stride, gate, gate_stride, out,      \
-                               out_stride, n_tokens, heads, dv, eps, stream);                                         \
+                                  const float* w, int w_head_stride, const T* gate, int64_t gate_stride,              \
+                                  int gate_silu, T* out, int64_t out_stride, int n_tokens, int heads, int dv,         \
+                                  float eps, cudaStream_t stream) {                                                   \
+    return head_norm_launch<T>(o, o_stride, o_cols, with_den, den_eps, w, w_head_stride, gate, gate_stride,           \
+                               gate_silu, out, out_stride, n_tokens, heads, dv, eps, stream);                                         \
   }                                                                                                                   \
   GLLM_API int gllm_gated_group_norm_##S(const float* y, int64_t y_stride, const T* x, int64_t x_stride,              \
                                          const float* skip, int head_width, const T* z, int64_t z_stride,             \

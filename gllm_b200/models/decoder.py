@@ -14,10 +14,12 @@ import torch
 from gllm_b200 import ops
 from gllm_b200.models.spec import ModelSpec
 from gllm_b200.parts import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, build_part
-from gllm_b200.parts.base import Block, MixerCache, Norm, StepContext, TensorExpectation
+from gllm_b200.parts.base import (DEPTH_AVERAGES, INPUT_CONVS, Block, MixerCache, Norm, StateRequirement, StepContext,
+                                  TensorExpectation)
 
 
-_TABLE_OF_KIND = {"mixer": MIXERS, "feed_forward": FEED_FORWARDS, "norm": NORMS}
+_TABLE_OF_KIND = {"mixer": MIXERS, "feed_forward": FEED_FORWARDS, "norm": NORMS, "input_conv": INPUT_CONVS,
+                  "depth_average": DEPTH_AVERAGES}
 
 
 def _build_layer(layer_spec) -> Block:
@@ -109,11 +111,15 @@ class DecoderModel:
         reads_cache_of | None)."""
         out = []
         for entry in self.spec.plan:
-            mixer = self.layers[entry.layer].cache_mixer()
-            if mixer is None:
-                out.append((None, None, entry.reads_cache_of))
-            else:
-                out.append((mixer.kv_requirement(), mixer.state_requirement(), entry.reads_cache_of))
+            block = self.layers[entry.layer]
+            mixer, extra = block.cache_mixer(), tuple(block.block_states())
+            if extra and entry.reads_cache_of is not None:
+                raise ValueError("an entry that reads another's cache cannot keep states of its own")
+            kv, state = (None, None) if mixer is None else (mixer.kv_requirement(), mixer.state_requirement())
+            if extra:
+                own = () if state is None else (state,) if isinstance(state, StateRequirement) else tuple(state)
+                state = own + extra
+            out.append((kv, state, entry.reads_cache_of))
         return out
 
     def kernel_needs(self) -> dict:
@@ -153,8 +159,15 @@ class DecoderModel:
             resid = stateful.embed_streams(tokens, self.embedding, ctx.positions, self._sinusoid_frequencies(),
                                            streams=self.spec.residual_streams, sampled=ctx.sampled,
                                            token_row=ctx.token_row, scale=scale)
+        elif self.spec.depth_streams:
+            # every layer's result is kept beside the embedding output until the step is over
+            ctx.depth_streams = torch.empty((len(self.spec.plan) + 1, tokens.numel(), self.spec.hidden_size),
+                                            dtype=torch.float32, device=self.device)
+            resid = ops.embedding(tokens, self.embedding, out=ctx.depth_streams[0], sampled=ctx.sampled,
+                                  token_row=ctx.token_row, scale=scale)
         else:
             resid = ops.embedding(tokens, self.embedding, sampled=ctx.sampled, token_row=ctx.token_row, scale=scale)
+        ctx.shared = {}
         branch = None
         first = None
         if any(entry.rejoins_embedding or entry.adds_embedding for entry in self.spec.plan):

@@ -95,11 +95,16 @@ class ModelSpec:
     # Checkpoint name of the ``[hidden, 2 * hidden]`` matrix of the plan entries that rejoin the embedding
     # (``PlanEntry.rejoins_embedding``); None when no entry does.
     rejoin_name: str | None = None
+    # The layers average over the depth of the model (blocks with a ``depth_average`` part): the embedding output and
+    # every layer's result are kept for the length of a step.
+    depth_streams: bool = False
     # Tensor names that a checkpoint may hold and the model does not read
     # (for instance a stored head beside tied embeddings).
     ignorable_names: tuple[str, ...] = ()
 
     def validate(self) -> None:
+        if self.depth_streams and (self.residual_streams != 1 or self.position_sinusoid_base is not None):
+            raise ValueError("an average over the depth is defined for a single residual stream without a sinusoid")
         for i, entry in enumerate(self.plan):
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(f"plan entry {i} names layer {entry.layer}, the model has {len(self.layers)}")

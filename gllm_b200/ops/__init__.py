@@ -50,6 +50,8 @@ __all__ = [
     "Pending",
     "rope_norm_store",
     "add_dyt",
+    "Biased",
+    "DepthPending",
 ]
 
 P = c_void_p
@@ -88,7 +90,7 @@ _SIGNATURES = {
         "gllm_gated_group_norm_{t}": [P, c_int64, P, c_int64, P, c_int, P, c_int64, P, P, c_int64, c_int, c_int, c_int,
                                       c_float, P],
         "gllm_conv_state_advance_{t}": [P, c_int64, P, P, P, c_int, c_int, c_int, P],
-        "gllm_head_norm_{t}": [P, c_int64, c_int, c_int, c_float, P, c_int, P, c_int64, P, c_int64, c_int, c_int,
+        "gllm_head_norm_{t}": [P, c_int64, c_int, c_int, c_float, P, c_int, P, c_int64, c_int, P, c_int64, c_int, c_int,
                                c_int, c_float, P],
     },
     "hyper_streams": {
@@ -103,7 +105,8 @@ _SIGNATURES = {
     },
     "attention_latent": {
         "gllm_latent_prep_{t}": [P, c_int64, P, c_int, c_int64, c_int, P, c_float, P, P, P, P, c_int, c_int, c_int, c_int,
-                                 c_int, c_int, c_int, c_int, c_int, c_int, P, P],
+                                 c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, P, P, P],
+        "gllm_latent_rotate_q_{t}": [P, c_int64, P, P, c_int, c_int, c_int, c_int, c_int, P],
         "gllm_head_linear_{t}": [P, c_int64, c_int, P, P, c_int64, c_int, c_int, c_int, c_int, c_int, P],
         "gllm_attention_latent_{t}": [P, c_int64, c_int, P, c_int64, c_int, P, c_int64, P, c_int64, c_int, P, P, c_int,
                                       P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, P, P],
@@ -117,6 +120,18 @@ _SIGNATURES = {
         "gllm_attention_diff_{t}": [P, c_int64, P, c_int64, P, c_int64, P, P, c_int, P, P, c_int, c_int, c_int, c_int,
                                     c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_float, P, P],
     },
+    "attention_distance": {
+        "gllm_distance_prep_{t}": [P, c_int64, P, c_int, c_int64, P, c_float, P, P, c_int, c_float, P, P, c_int, c_int,
+                                   c_int, c_int, c_int, c_int, c_int, P, P],
+        "gllm_attention_distance_{t}": [P, c_int64, P, c_int64, P, P, c_int, P, P, P, c_int, P, c_int, c_int, c_int,
+                                        c_int, c_int, c_int, c_int, c_float, c_int, c_int, P, P],
+    },
+    "depth_conv": {
+        "gllm_depth_conv_{t}": [P, P, c_int, c_int64, P, P, c_float, P, P, c_int64, c_int, P, P, P, P, P, P, P, c_int,
+                                c_int, c_int, c_int, P],
+        "gllm_depth_norm_{t}": [P, P, c_int, c_int64, P, P, c_float, P, P, c_int64, c_int, P, P, c_int, P, c_float, P,
+                                c_int, P],
+    },
     "postnorm": {
         "gllm_postnorm_add_rmsnorm_{t}": [P, P, c_int, c_int64, P, c_float, P, P, P, c_float, P, P, c_int, c_int, P],
     },
@@ -126,8 +141,8 @@ _SIGNATURES = {
     },
     "delta_rule": {
         "gllm_delta_prep_{t}": [P, c_int64, P, P, P, P, P, P, c_int, P, c_int64, P, P, P, c_int64, P, P, P, P, c_int,
-                                c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, P],
-        "gllm_delta_rule": [P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P],
+                                c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, P],
+        "gllm_delta_rule": [P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P],
     },
     "moe": {
         "gllm_moe_route": [P, c_int64, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
@@ -368,6 +383,27 @@ class Pending:
         return Pending(self.value, self.post_weight, self.post_eps, extra)
 
 
+class Biased:
+    """The result of a branch's last product (a tensor or a SplitSum) whose bias (fp32, one value per column) has not
+    been added yet: for blocks whose next kernel adds it (``StepContext.takes_bias``)."""
+
+    def __init__(self, value, bias: torch.Tensor):
+        self.value, self.bias = value, bias
+
+
+class DepthPending:
+    """What is still to be done to the fp32 residual when the next norm runs: ``value`` (a tensor of the activation type
+    or a SplitSum, with ``value_bias`` still to be added) is RMS-normed with ``post_weight`` and ``post_eps`` and added;
+    with ``depth_weight`` (fp32 ``[count + 1]``) the sum ``X`` is then replaced by the weighted sum over ``streams
+    [>= count + 1, n, width]`` (fp32: ``count`` earlier streams and a place for ``X``).  ``value`` None: nothing is
+    added."""
+
+    def __init__(self, value=None, value_bias=None, post_weight=None, post_eps: float = 0.0, streams=None,
+                 count: int = 0, depth_weight=None):
+        self.value, self.value_bias, self.post_weight, self.post_eps = value, value_bias, post_weight, float(post_eps)
+        self.streams, self.count, self.depth_weight = streams, int(count), depth_weight
+
+
 def _parts_args(x):
     if isinstance(x, SplitSum):
         x.check_alive()
@@ -474,6 +510,12 @@ def add_rmsnorm(
     hidden = resid.shape[-1]
     if weight.numel() != hidden:
         raise ValueError(f"norm weight has {weight.numel()} elements, rows have {hidden}")
+    if isinstance(branch, DepthPending):
+        from gllm_b200.ops import depth
+
+        if unit_offset or out is not None:
+            raise ValueError("a norm over a depth average takes a plain weight and makes its own result")
+        return depth.depth_norm(branch, resid, weight, eps, out_dtype, rows)
     if isinstance(branch, Pending):
         if branch.post_weight is None and branch.extra is None:
             branch = branch.value

@@ -61,6 +61,9 @@ MODULES = {
     "dyt_norm": "dyt_norm.cu",
     "attention_diff": "attention_diff.cu",
     "attention_diff_mma": "attention_diff_mma.cu",
+    "attention_distance": "attention_distance.cu",
+    "attention_distance_mma": "attention_distance_mma.cu",
+    "depth_conv": "depth_conv.cu",
 }
 
 _loaded: dict[str, ctypes.CDLL] = {}

@@ -26,7 +26,7 @@ def _mma_fns():
         f = lib.gllm_attention_latent_mma
         P = c_void_p
         f.argtypes = [P, c_int64, P, c_int64, c_int, P, c_int64, P, c_int64, P, P, P, P, c_int, P, P, P, c_int, c_int,
-                      c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, P, P]
+                      c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, P, P]
         f.restype = c_int
         lib.gllm_attention_latent_mma_supports.argtypes = [c_int, c_int]
         lib.gllm_attention_latent_mma_supports.restype = c_int
@@ -39,16 +39,15 @@ def _mma_fns():
     return _mma
 
 
-MMA_SIZES = {(64, 32), (64, 64), (96, 32), (128, 32), (128, 64), (256, 32), (256, 64), (512, 64)}
-
-
 def tensor_core_kernel_takes(dtype: torch.dtype, rank: int, rot: int) -> bool:
-    """True for the (latent, rotated part) widths the tensor-core kernel is built for, in bfloat16."""
-    return dtype == torch.bfloat16 and (rank, rot) in MMA_SIZES and USE_TENSOR_CORES
+    """True for the (latent, rotated part) widths the tensor-core kernel takes, in bfloat16: multiples of 8 up to 512
+    and 64 (it is built for a few pairs of widths; narrower vectors fill part of a tile)."""
+    return (dtype == torch.bfloat16 and USE_TENSOR_CORES and 0 < rank <= 512 and 0 <= rot <= 64
+            and rank % 8 == 0 and rot % 8 == 0)
 
 
 def _attention_latent_mma(qa, rows, q_head, q_plain, gate_col, pages, block_table, heads, rank, rot, block_size, scale,
-                          batch, out):
+                          batch, out, window=0):
     """The tensor-core kernel.  Steps whose tiles do not fill the GPU (single tokens over long contexts) cut every
     request's keys into ranges of at least ``SPLIT_KEYS`` keys, one CTA each, merged by a second kernel."""
     f, _, tokens_per_tile = _mma_fns()[:3]
@@ -65,6 +64,8 @@ def _attention_latent_mma(qa, rows, q_head, q_plain, gate_col, pages, block_tabl
     longest = batch.max_seq_len
     if batch.max_q_len > 1 and torch.cuda.is_current_stream_capturing():
         longest = max(longest, block_table.shape[1] * block_size)
+    if window:              # a CTA visits what its first token's window holds and its own tokens, on whole tiles
+        longest = min(longest, window + qt + KEY_TILE)
     if 2 * tiles <= sms and longest > 2 * SPLIT_KEYS:
         want = min(MAX_SPLITS, -(-2 * sms // tiles))
         key_tiles = -(-longest // KEY_TILE)
@@ -80,7 +81,7 @@ def _attention_latent_mma(qa, rows, q_head, q_plain, gate_col, pages, block_tabl
              rows.stride(0), out.data_ptr(), out.stride(0), _ptr(part_o), _ptr(part_ml), pages.data_ptr(),
              block_table.data_ptr(), block_table.stride(0), batch.cu_q.data_ptr(), batch.context_lens.data_ptr(),
              batch.state_slots.data_ptr(), batch.num_requests, batch.max_q_len, n, int(heads), int(rank), int(rot),
-             int(block_size), pages.shape[0], float(scale), splits, tiles_per_split,
+             int(block_size), pages.shape[0], float(scale), int(window), splits, tiles_per_split,
              status_word(qa.device).data_ptr(), _stream())
     _check(code, "attention_latent_mma")
     return out
@@ -94,13 +95,15 @@ def _rows(t: torch.Tensor, name: str, dtype=None) -> None:
 
 def latent_prep(rows, norm_weight: torch.Tensor, eps: float, positions: torch.Tensor,
                 inv_freq: torch.Tensor, slot_mapping: torch.Tensor | None, pages: torch.Tensor, heads: int,
-                q_plain: int, rot: int, rank: int, down_col: int, block_size: int) -> torch.Tensor:
+                q_plain: int, rot: int, rank: int, down_col: int, block_size: int,
+                q_latent_norm: torch.Tensor | None = None):
     """On the projection rows ``[n, >= heads * (q_plain + rot) + rank + rot]`` (a tensor, or a SplitSum that is
     summed into a new tensor first, in the same kernel): rotate the last ``rot`` columns of every query head in
     place (neighbouring pairs, ``2 * len(inv_freq)`` columns of them), and store
     ``[rms(down[:rank]) * norm_weight ; rotate(down[rank:])]`` of the down-projection at column ``down_col``
     into the token's cache slot.  ``pages`` is the pool layer ``[pages, block_size * (rank + rot)]``.  Returns the
-    rows."""
+    rows.  With ``q_latent_norm`` (one weight per column of the queries' latent; ``heads`` 0: the rows hold no query
+    heads) returns ``rms(rows[:, :q_rank]) * q_latent_norm`` instead, ``[n, q_rank]``."""
     from gllm_b200.ops import SplitSum, _parts_args
 
     parts_ptr, n_parts, part_stride = _parts_args(rows)
@@ -123,11 +126,34 @@ def latent_prep(rows, norm_weight: torch.Tensor, eps: float, positions: torch.Te
         raise ValueError("the projection rows are narrower than the heads and the down-projection need")
     if slot_mapping is not None:
         _cuda(slot_mapping, "slot_mapping", torch.int32)
+    q_rank, q_latent = 0, None
+    if q_latent_norm is not None:
+        _cuda(q_latent_norm, "q_latent_norm", torch.float32)
+        q_rank = q_latent_norm.numel()
+        if heads or q_rank > down_col:
+            raise ValueError("rows that hold the queries' latent hold it before the down-projection and no query heads")
+        q_latent = torch.empty((rows.shape[0], q_rank), dtype=rows.dtype, device=rows.device)
     f = _fn("attention_latent", f"gllm_latent_prep_{_suffix(rows.dtype)}")
     _check(f(rows.data_ptr(), rows.stride(0), parts_ptr, n_parts, part_stride, rows.shape[1], norm_weight.data_ptr(),
              float(eps), positions.data_ptr(), inv_freq.data_ptr(), _ptr(slot_mapping), pages.data_ptr(), rows.shape[0],
              int(heads), int(q_plain + rot), int(q_plain), int(down_col), int(rank), int(rot), 2 * inv_freq.numel(),
-             int(block_size), pages.shape[0], status_word(rows.device).data_ptr(), _stream()), "latent_prep")
+             int(block_size), pages.shape[0], q_rank, _ptr(q_latent_norm), _ptr(q_latent),
+             status_word(rows.device).data_ptr(), _stream()), "latent_prep")
+    return rows if q_latent is None else q_latent
+
+
+def latent_rotate_q(rows: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, heads: int, q_plain: int,
+                    rot: int) -> torch.Tensor:
+    """Rotate neighbouring pairs of the first ``2 * len(inv_freq)`` columns of the rotated part (the last ``rot``
+    columns) of every query head of ``rows [n, heads * (q_plain + rot)]``, in place."""
+    _rows(rows, "rows")
+    _cuda(positions, "positions", torch.int32)
+    _cuda(inv_freq, "inv_freq", torch.float32)
+    if rows.shape[1] < heads * (q_plain + rot) or 2 * inv_freq.numel() > rot:
+        raise ValueError("the rows are narrower than the heads need")
+    f = _fn("attention_latent", f"gllm_latent_rotate_q_{_suffix(rows.dtype)}")
+    _check(f(rows.data_ptr(), rows.stride(0), positions.data_ptr(), inv_freq.data_ptr(), rows.shape[0], int(heads),
+             int(q_plain + rot), int(q_plain), inv_freq.numel(), _stream()), "latent_rotate_q")
     return rows
 
 
@@ -160,7 +186,7 @@ def attention_latent(qa: torch.Tensor, rows: torch.Tensor, q_head: int, q_plain:
                      batch=None) -> torch.Tensor:
     """Softmax attention of every (token, head) over its request's cached ``[c ; kr]`` vectors: scores
     ``(qa . c + qr . kr) * scale`` with ``qa [n, heads * rank]`` and ``qr`` the rotated part of every query head
-    inside ``rows``; the result ``[n, heads * rank]`` is the weighted sum of the ``c`` (times
+    inside ``rows``, over the keys less than ``window`` positions back when one is given; the result ``[n, heads * rank]`` is the weighted sum of the ``c`` (times
     ``sigmoid(rows[n, gate_col + h])`` with ``gate_col``)."""
     _rows(qa, "qa")
     _rows(rows, "rows", qa.dtype)
@@ -172,11 +198,11 @@ def attention_latent(qa: torch.Tensor, rows: torch.Tensor, q_head: int, q_plain:
     if qa.shape[1] != heads * rank or pages.stride(0) != block_size * (rank + rot):
         raise ValueError("qa or the cache layer does not match heads, rank and rot")
     out = torch.empty((n, heads * rank), dtype=qa.dtype, device=qa.device)
-    if (batch is not None and not window and tensor_core_kernel_takes(qa.dtype, rank, rot) and qa.stride(0) % 8 == 0
+    if (batch is not None and tensor_core_kernel_takes(qa.dtype, rank, rot) and qa.stride(0) % 8 == 0
             and rows.stride(0) % 8 == 0 and q_head % 8 == 0 and q_plain % 8 == 0
             and rows.data_ptr() % 16 == 0 and qa.data_ptr() % 16 == 0):
         return _attention_latent_mma(qa, rows, q_head, q_plain, gate_col, pages, block_table, heads, rank, rot,
-                                     block_size, scale, batch, out)
+                                     block_size, scale, batch, out, window=int(window or 0))
     t = _suffix(qa.dtype)
     item = qa.element_size()
     f = _fn("attention_latent", f"gllm_attention_latent_{t}")

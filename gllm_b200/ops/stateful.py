@@ -250,10 +250,10 @@ def conv_state_advance(x: torch.Tensor, conv_state: torch.Tensor, cu_q: torch.Te
 
 def head_norm(o: torch.Tensor, heads: int, dv: int, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
               with_denominator: bool = False, denominator_eps: float = 0.0,
-              gate: torch.Tensor | None = None) -> torch.Tensor:
+              gate: torch.Tensor | None = None, gate_kind: str = "sigmoid") -> torch.Tensor:
     """Each head of ``o`` (fp32 ``[n, heads * cols]`` as ``matrix_recurrence`` returns it) divided by
     its root mean square over its ``dv`` values, times ``weight`` (``[dv]``: shared by the heads;
-    ``[heads * dv]``: one per column), times ``sigmoid(gate)`` when given.  ``with_denominator``: the
+    ``[heads * dv]``: one per column), times ``sigmoid(gate)`` (or ``silu(gate)``, ``gate_kind`` "silu") when given.  ``with_denominator``: the
     head is first divided by ``max(|o[dv]|, o[dv+1]) + denominator_eps``."""
     _cuda(o, "o", torch.float32)
     _cuda(weight, "weight", torch.float32)
@@ -261,14 +261,16 @@ def head_norm(o: torch.Tensor, heads: int, dv: int, weight: torch.Tensor, eps: f
     cols = o.shape[1] // heads
     if weight.numel() not in (dv, heads * dv) or cols < dv + (2 if with_denominator else 0):
         raise ValueError("head_norm's operands do not fit together")
+    if gate_kind not in ("sigmoid", "silu"):
+        raise ValueError(f"unknown gate {gate_kind!r}")
     if gate is not None:
         _rows(gate, "gate", out_dtype)
     out = torch.empty((n, heads * dv), dtype=out_dtype, device=o.device)
     f = _fn("recurrent", f"gllm_head_norm_{_suffix(out_dtype)}")
     _check(f(o.data_ptr(), o.stride(0), cols, int(with_denominator), float(denominator_eps), weight.data_ptr(),
              dv if weight.numel() == heads * dv and heads > 1 else 0, _ptr(gate),
-             gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), n, heads, dv, float(eps),
-             _stream()), "head_norm")
+             gate.stride(0) if gate is not None else 0, int(gate_kind == "silu"), out.data_ptr(), out.stride(0), n, heads,
+             dv, float(eps), _stream()), "head_norm")
     return out
 
 
@@ -283,10 +285,11 @@ def delta_prep(x: torch.Tensor, conv_weight: torch.Tensor, conv_state: torch.Ten
     heads * dv``; each channel passes a causal convolution over the request's own tokens (``conv_weight
     [channels, taps]`` fp32, last column = the current token; ``conv_state [slots, taps-1, channels]`` fp32 holds
     every request's last inputs, oldest first, and is brought up to date) and SiLU; every q and k head becomes
-    ``x / sqrt(sum(x^2) + unit_eps)``, q also times ``q_scale``.  ``decay_raw [n, heads * dk]`` and ``beta_raw
-    [n, heads]`` are fp32: ``g = exp(-exp(A_log[h]) * softplus(decay_raw + dt_bias))``, ``beta = sigmoid(beta_raw)``.
+    ``x / sqrt(sum(x^2) + unit_eps)``, q also times ``q_scale``.  ``decay_raw [n, heads * dk]`` (a decay per key channel;
+    ``[n, heads]``: one per head) and ``beta_raw [n, heads]`` are fp32, rows may be slices: ``g = exp(-exp(A_log[h]) *
+    softplus(decay_raw + dt_bias))``, ``beta = sigmoid(beta_raw)``.
     ``max_q_len`` 1 says that every request brings one token: the state is then brought up to date by the same
-    kernel.  Returns ``(qk [n, 2 * kv_heads * dk], v [n, heads * dv], g [n, heads * dk], beta [n, heads])``."""
+    kernel.  Returns ``(qk [n, 2 * kv_heads * dk], v [n, heads * dv], g [n, heads * dk or heads], beta [n, heads])``."""
     _rows(x, "x")
     _rows(decay_raw, "decay_raw", torch.float32)
     _rows(beta_raw, "beta_raw", torch.float32)
@@ -295,28 +298,29 @@ def delta_prep(x: torch.Tensor, conv_weight: torch.Tensor, conv_state: torch.Ten
     n = x.shape[0]
     qk_cols, channels = 2 * kv_heads * dk, 2 * kv_heads * dk + heads * dv
     taps = conv_weight.shape[1]
+    decay_width = 1 if decay_raw.shape[1] == heads else dk
     if (x.shape[1] < channels or conv_weight.shape[0] != channels
-            or tuple(conv_state.shape[1:]) != (max(taps - 1, 0), channels) or decay_raw.shape[1] != heads * dk
-            or beta_raw.shape[1] != heads or dt_bias.numel() != heads * dk or A_log.numel() != heads):
+            or tuple(conv_state.shape[1:]) != (max(taps - 1, 0), channels) or decay_raw.shape[1] != heads * decay_width
+            or beta_raw.shape[1] != heads or dt_bias.numel() != heads * decay_width or A_log.numel() != heads):
         raise ValueError("the delta rule's operands do not fit together")
     dev = x.device
     qk = torch.empty((n, qk_cols), dtype=torch.float32, device=dev)
     v = torch.empty((n, heads * dv), dtype=torch.float32, device=dev)
-    g = torch.empty((n, heads * dk), dtype=torch.float32, device=dev)
+    g = torch.empty((n, heads * decay_width), dtype=torch.float32, device=dev)
     beta = torch.empty((n, heads), dtype=torch.float32, device=dev)
     f = _fn("delta_rule", f"gllm_delta_prep_{_suffix(x.dtype)}")
     _check(f(x.data_ptr(), x.stride(0), conv_weight.data_ptr(), conv_state.data_ptr(), positions.data_ptr(),
              token_row.data_ptr(), cu_q.data_ptr(), state_slots.data_ptr(), int(num_requests), decay_raw.data_ptr(),
              decay_raw.stride(0), dt_bias.data_ptr(), A_log.data_ptr(), beta_raw.data_ptr(), beta_raw.stride(0),
              qk.data_ptr(), v.data_ptr(), g.data_ptr(), beta.data_ptr(), n, heads, kv_heads, dk, dv, taps,
-             float(unit_eps), float(q_scale), int(max_q_len), _stream()), "delta_prep")
+             float(unit_eps), float(q_scale), int(max_q_len), decay_width, _stream()), "delta_prep")
     return qk, v, g, beta
 
 
 def delta_rule(qk: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
                cu_q: torch.Tensor, state_slots: torch.Tensor, num_requests: int, heads: int, kv_heads: int, dk: int,
                dv: int, max_q_len: int = 0) -> torch.Tensor:
-    """Per (request, head), token after token: ``S <- diag(g) S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
+    """Per (request, head), token after token: ``S <- diag(g) S`` (``g`` a number per key channel, or per head), ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
     ``o = S^T q`` (the read-out sees the token's own write).  Operands as ``delta_prep`` returns them; head ``h``
     uses the q and k of head ``h // (heads / kv_heads)``.  ``state [slots, heads, dv, dk]`` fp32 (one row per value
     column) is updated in place.  Returns fp32 ``[n, heads * dv]``."""
@@ -324,13 +328,14 @@ def delta_rule(qk: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.T
         _cuda(t, name, torch.float32)
     n = qk.shape[0]
     if (tuple(state.shape[1:]) != (heads, dv, dk) or qk.shape[1] != 2 * kv_heads * dk or v.shape[1] != heads * dv
-            or g.shape[1] != heads * dk or beta.shape[1] != heads):
+            or g.shape[1] not in (heads * dk, heads) or beta.shape[1] != heads):
         raise ValueError("the delta rule's operands do not fit together")
+    decay_width = 1 if g.shape[1] == heads else dk
     out = torch.empty((n, heads * dv), dtype=torch.float32, device=qk.device)
     f = _fn("delta_rule", "gllm_delta_rule")
     _check(f(qk.data_ptr(), v.data_ptr(), g.data_ptr(), beta.data_ptr(), state.data_ptr(), cu_q.data_ptr(),
              state_slots.data_ptr(), out.data_ptr(), int(num_requests), heads, kv_heads, dk, dv, int(max_q_len),
-             _stream()), "delta_rule")
+             decay_width, _stream()), "delta_rule")
     return out
 
 

@@ -2,7 +2,7 @@
 
 A part knows its own sizes and constants (constructor parameters) and the
 checkpoint names of its tensors; it never sees a model configuration and does
-not know which model it is in.  Five kinds exist:
+not know which model it is in.  Seven kinds exist:
 
 * ``Mixer``            mixes information between the tokens of a request
                        (attention here); may keep keys and values in cache
@@ -12,7 +12,11 @@ not know which model it is in.  Five kinds exist:
 * ``Norm``             normalises the residual stream before a mixer or a
                        feed-forward, fused with the residual add;
 * ``PositionEncoding`` tells a mixer how positions enter;
-* ``Block``            the arrangement of the four above in one layer.
+* ``InputConv``        convolves what a sublayer reads over time (keeps its last
+                       inputs per request);
+* ``DepthAverage``     replaces the residual after a layer by a weighted sum over
+                       the embedding output and all layers' results;
+* ``Block``            the arrangement of those above in one layer.
 
 The reference has one fixed class for each (gllm/model/layers/attention.py,
 mlp.py, norm.py, gllm/model/transformer.py) that pulls its tensors out of the
@@ -56,8 +60,10 @@ class KVPageRequirement:
     other, each as ``[heads, block_size, width]``."""
 
     tensors: tuple[tuple[int, int], ...]
-    # None: all tokens stay.  w: a token at position p needs positions > p - w.
+    # None: all tokens stay.  w: a token at position p needs positions > p - w ...
     window: int | None = None
+    # ... and, for as long as the request lives, the positions below this one
+    keep_first: int = 0
 
     def __post_init__(self):
         if not self.tensors or any(len(t) != 2 or t[0] <= 0 or t[1] <= 0 for t in self.tensors):
@@ -131,6 +137,14 @@ class StepContext:
     # and return what that returns (``ops.ADDED`` when the product added itself); parts that ignore
     # it return their result as before.
     residual_sink: Any = None
+    # Set by a block around a part's call: the part may leave its last product's bias to the block's next kernel and
+    # return ``ops.Biased(value, bias)``.
+    takes_bias: bool = False
+    # what a layer leaves for later layers of the same step (key -> tensor over the step's tokens)
+    shared: dict = field(default_factory=dict)
+    # fp32 [plan entries + 1, n, hidden] of a model that averages over its depth: the embedding output, then every
+    # layer's result as it is made
+    depth_streams: Any = None
 
 
 @dataclass
@@ -143,7 +157,8 @@ class MixerCache:
     state: torch.Tensor | None = None     # [max_batch_size + 1, *StateRequirement.shape]; last row: padding rows
     requirement: KVPageRequirement | None = None
     block_size: int = 0
-    # every state tensor the mixer declared, in its order (``state`` is the first of them)
+    # every state tensor the plan entry's mixer declared, in its order (``state`` is the first of them), then those
+    # its block declared
     states: tuple = ()
 
     def tensor(self, index: int) -> torch.Tensor:
@@ -235,13 +250,29 @@ class FeedForward(Part):
         raise NotImplementedError
 
 
+class InputConv(Part):
+    """A causal convolution over time of what a sublayer reads; ``weight`` is fp32 ``[taps, width]`` (last row: the
+    current token) once loaded."""
+
+    weight: "torch.Tensor | None" = None
+
+    def state_requirement(self) -> StateRequirement:
+        raise NotImplementedError
+
+
+class DepthAverage(Part):
+    """``weight``: fp32, one number per stream (the embedding output, then one per layer run so far)."""
+
+    weight: "torch.Tensor | None" = None
+
+
 class Block(Part):
     """Arrangement of a layer's parts.  ``forward`` gets the previous layer's
     not yet added branch output and the fp32 residual stream, and returns its
     own last branch output with the (updated in place) residual stream.
 
     A block kind declares the parts it is made of in ``part_kinds``: part name
-    -> "mixer" | "feed_forward" | "norm", in the order they are loaded.  The
+    -> "mixer" | "feed_forward" | "norm" | "input_conv" | "depth_average", in the order they are loaded.  The
     decoder builds exactly those from a ``LayerSpec`` and hands them to the
     constructor by name; each becomes an attribute.  A block holds at most one
     mixer that asks for a cache (the plan gives every entry one cache)."""
@@ -271,6 +302,11 @@ class Block(Part):
             raise ValueError("a block holds at most one mixer")
         return mixers[0] if mixers else None
 
+    def block_states(self) -> tuple[StateRequirement, ...]:
+        """State tensors per request that the block keeps beside its mixer's (they follow the mixer's in
+        ``MixerCache.states``)."""
+        return ()
+
     def forward(self, branch, resid, ctx: StepContext, cache: MixerCache):
         raise NotImplementedError
 
@@ -280,6 +316,8 @@ MIXERS: dict[str, type] = {}
 FEED_FORWARDS: dict[str, type] = {}
 NORMS: dict[str, type] = {}
 POSITION_ENCODINGS: dict[str, type] = {}
+INPUT_CONVS: dict[str, type] = {}
+DEPTH_AVERAGES: dict[str, type] = {}
 BLOCKS: dict[str, type] = {}
 
 
@@ -306,6 +344,14 @@ def register_norm(kind: str):
 
 def register_position_encoding(kind: str):
     return _register(POSITION_ENCODINGS, kind)
+
+
+def register_input_conv(kind: str):
+    return _register(INPUT_CONVS, kind)
+
+
+def register_depth_average(kind: str):
+    return _register(DEPTH_AVERAGES, kind)
 
 
 def register_block(kind: str):

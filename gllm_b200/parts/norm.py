@@ -33,6 +33,16 @@ class RMSNorm(Norm):
     def load(self, get, dtype, device):
         self.weight = get(self.names["weight"], "vector")
 
+    def depth_pending(self, value, streams=None, count: int = 0, depth_weight=None):
+        """``value`` (a sublayer's result, possibly ``ops.Biased``) as an ``ops.DepthPending`` with this norm's weight,
+        for blocks whose next kernel norms it, adds it and averages over the depth."""
+        if self.unit_offset:
+            raise ValueError("a norm whose weight is stored around zero cannot follow a sublayer")
+        bias = None
+        if isinstance(value, ops.Biased):
+            value, bias = value.value, value.bias
+        return ops.DepthPending(value, bias, self.weight, self.eps, streams, count, depth_weight)
+
     def pending(self, value):
         """``value`` (a sublayer's result) as what the NEXT norm's kernel norms with this norm's weight and adds
         to the residual: the norm after a sublayer of a layer that norms both sides of it."""
