@@ -592,7 +592,29 @@ def sazisun_raw(sz: dict) -> dict:
             "layers": layers, "torch_dtype": "bfloat16"}
 
 
-DESIGNS = {"guvetar": guvetar_raw, "rulunex": rulunex_raw, "mifidra": mifidra_raw, "sazisun": sazisun_raw}
+def vonedra_raw(sz: dict) -> dict:
+    """``layers`` layers: attention with a bias by distance, latent attention and the delta rule in turn, each with a
+    dense feed-forward of Llama's width; both attentions see a window of 1,024 tokens, the first also the first 64."""
+    attention = {"type": "attention", "mixer": {
+        "heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": sz["head_dim"], "vdim": sz["head_dim"],
+        "scale": sz["head_dim"] ** -0.5, "bias_max": 1000, "bias_rows": 32, "v_mix": True,
+        "mask": {"size": 1024, "keep_first": 64}}}
+    latent = {"type": "latent_attention", "mixer": {
+        "heads": sz["latent_heads"], "dim": sz["latent_dim"], "rot_dim": sz["latent_rot"], "vdim": sz["latent_dim"],
+        "q_rank": sz["width"] * 3 // 8, "kv_rank": sz["latent_rank"],
+        "scale": (sz["latent_dim"] + sz["latent_rot"]) ** -0.5, "mask": {"size": 1024},
+        "rot": {"base": 10000.0, "dims": sz["latent_rot"]}}}
+    delta = {"type": "delta", "mixer": {"heads": sz["linear_heads"], "kv_heads": sz["linear_heads"],
+                                        "dim": sz["linear_dim"], "vdim": sz["linear_vdim"], "conv": 4}}
+    kinds = [attention, latent, delta]
+    return {"architecture": "Vonedra", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": 8.0}, "canon": {"taps": 4},
+            "layers": [{**kinds[i % 3], "mlp": {"kind": "dense", "ff": sz["ff"]}} for i in range(sz["layers"])],
+            "torch_dtype": "bfloat16"}
+
+
+DESIGNS = {"guvetar": guvetar_raw, "rulunex": rulunex_raw, "mifidra": mifidra_raw, "sazisun": sazisun_raw,
+           "vonedra": vonedra_raw}
 
 
 def llama_raw(sz: dict) -> dict:

@@ -259,6 +259,13 @@ def _result(name, us, peaks, shape, nbytes=None, flops=None):
     return out
 
 
+def _visible(tokens, context, window=0, keep=0):
+    """(query, key) pairs of one request: every query sees ``window`` keys and the first ``keep`` beside them."""
+    if not window:
+        return tokens * context + tokens * (tokens + 1) / 2
+    return float(sum(min(p + 1, window) + min(keep, max(0, p + 1 - window)) for p in range(context, context + tokens)))
+
+
 def sigmoid_attention(tokens=2048, batch=1, context=0, hq=32, hkv=8, dk=64, dv=64, block_size=16, iters=5, peaks=None,
                       mma=1):
     """``batch`` requests of ``tokens`` new tokens over ``context`` cached ones (tokens=1: a decode step)."""
@@ -284,10 +291,10 @@ def sigmoid_attention(tokens=2048, batch=1, context=0, hq=32, hkv=8, dk=64, dv=6
 
 
 def latent_attention(tokens=2048, batch=1, context=0, heads=16, rank=512, rot=64, block_size=16, iters=5, peaks=None,
-                     mma=1, split_keys=0):
+                     mma=1, split_keys=0, window=0):
     """``batch`` requests of ``tokens`` new tokens over ``context`` cached ones (tokens=1: a decode step) through
-    the latent attention kernel (with its merge when the keys are cut into ranges).  FLOPs: both products over the
-    visible keys; bytes: every request's cached vectors once, the queries and the result."""
+    the latent attention kernel (with its merge when the keys are cut into ranges), over all keys or a ``window``.
+    FLOPs: both products over the visible keys; bytes: every request's cached vectors once, the queries and the result."""
     from gllm_b200.ops import latent
 
     latent.USE_TENSOR_CORES = bool(mma)
@@ -305,12 +312,13 @@ def latent_attention(tokens=2048, batch=1, context=0, heads=16, rank=512, rot=64
     b = _Batch(batch, tokens, context)
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
     fn = lambda: latent.attention_latent(qa, rows, q_head, 128, heads * q_head, pool, table, b.positions, b.token_row,
-                                         heads, rank, rot, block_size, dk ** -0.5, batch=b)
+                                         heads, rank, rot, block_size, dk ** -0.5, window=window or None, batch=b)
     us = _time(fn, iters, flush)
-    flops = 2.0 * (dk + rank) * heads * batch * (tokens * context + tokens * (tokens + 1) / 2)
-    nbytes = batch * (context + tokens) * dk * 2 + qa.numel() * 4 + batch * tokens * heads * rot * 2
+    flops = 2.0 * (dk + rank) * heads * batch * _visible(tokens, context, window)
+    nbytes = batch * min(context + tokens, window + tokens if window else 1 << 30) * dk * 2 + qa.numel() * 4 + batch * tokens * heads * rot * 2
     return _result("latent_attention (mma.sync)" if mma else "latent_attention (CUDA cores)", us, peaks,
-                   dict(tokens=tokens, batch=batch, context=context, heads=heads, rank=rank, rot=rot), nbytes, flops)
+                   dict(tokens=tokens, batch=batch, context=context, heads=heads, rank=rank, rot=rot, window=window),
+                   nbytes, flops)
 
 
 def head_linear(tokens=2048, heads=16, inner=128, outer=512, iters=5, peaks=None, mma=1):
@@ -402,9 +410,9 @@ def stream_mix_norm(rows=2048, hidden=2048, streams=4, iters=5, peaks=None):
                    rows * hidden * (8 * streams + 4))
 
 
-def delta_rule(tokens=2048, batch=1, heads=16, dk=64, dv=128, taps=4, prep=0, iters=5, peaks=None):
-    """The gated delta rule's recurrence over ``batch`` requests of ``tokens`` tokens (tokens=1: a decode step);
-    ``prep=1`` times the kernel before it instead (convolution, SiLU, unit norms, decays, beta)."""
+def delta_rule(tokens=2048, batch=1, heads=16, dk=64, dv=128, taps=4, prep=0, head=0, iters=5, peaks=None):
+    """The gated delta rule's recurrence over ``batch`` requests of ``tokens`` tokens (tokens=1: a decode step), with a
+    decay per key channel or (``head=1``) one per head; ``prep=1`` times the kernel before it instead (convolution, SiLU, unit norms, decays, beta)."""
     from gllm_b200.ops import stateful
 
     n = batch * tokens
@@ -415,21 +423,22 @@ def delta_rule(tokens=2048, batch=1, heads=16, dk=64, dv=128, taps=4, prep=0, it
     x = torch.randn(n, channels, device="cuda").to(torch.bfloat16)
     conv_w = torch.randn(channels, taps, device="cuda") * 0.5
     conv_state = torch.zeros(batch + 1, taps - 1, channels, device="cuda")
-    raw, braw = torch.randn(n, heads * dk, device="cuda"), torch.randn(n, heads, device="cuda")
-    dt_bias, A_log = torch.zeros(heads * dk, device="cuda"), torch.full((heads,), -3.0, device="cuda")
+    dw = 1 if head else dk
+    raw, braw = torch.randn(n, heads * dw, device="cuda"), torch.randn(n, heads, device="cuda")
+    dt_bias, A_log = torch.zeros(heads * dw, device="cuda"), torch.full((heads,), -3.0, device="cuda")
     run_prep = lambda: stateful.delta_prep(x, conv_w, conv_state, b.positions, b.token_row, b.cu_q, b.state_slots, batch,
                                            raw, dt_bias, A_log, braw, heads, heads, dk, dv, 1e-6, dk ** -0.5)
     if prep:
         us = _time(run_prep, iters, flush)
-        nbytes = n * (channels * 2 + heads * dk * 4 + heads * 4) + n * (channels + heads * dk + heads) * 4
+        nbytes = n * (channels * 2 + heads * dw * 4 + heads * 4) + n * (channels + heads * dw + heads) * 4
         return _result("delta_prep", us, peaks, dict(shape, taps=taps), nbytes)
     qk, v, g, beta = run_prep()
     state = torch.zeros(batch + 1, heads, dv, dk, device="cuda")
     fn = lambda: stateful.delta_rule(qk, v, g, beta, state, b.cu_q, b.state_slots, batch, heads, heads, dk, dv,
                                      max_q_len=tokens)
     us = _time(fn, iters, flush)
-    nbytes = 2 * batch * heads * dk * dv * 4 + n * heads * (3 * dk + 2 * dv + 1) * 4
-    return _result("delta_rule", us, peaks, shape, nbytes, 6.0 * n * heads * dk * dv)
+    nbytes = 2 * batch * heads * dk * dv * 4 + n * heads * (2 * dk + dw + 2 * dv + 1) * 4
+    return _result("delta_rule (decay per head)" if head else "delta_rule", us, peaks, shape, nbytes, 6.0 * n * heads * dk * dv)
 
 
 def routed_experts(tokens=2048, width=2048, ff=1024, experts=16, top=4, groups=4, keep=3, mma=1, iters=5, peaks=None):
@@ -549,7 +558,72 @@ def ungated_experts(tokens=2048, width=2048, ff=2048, experts=16, top=4, groups=
                    4.0 * tokens * top * ff * width)
 
 
+def distance_attention(tokens=2048, batch=1, context=0, hq=32, hkv=8, dk=64, dv=64, window=0, keep=0, block_size=16,
+                       iters=5, peaks=None, mma=1, prep=0):
+    """``batch`` requests of ``tokens`` new tokens over ``context`` cached ones (tokens=1: a decode step): attention with
+    a bias by distance and a sink, over all keys or a ``window`` and the first ``keep``; ``prep=1`` times the kernel
+    before it instead (biases, norms, mix of the values, store)."""
+    from gllm_b200.ops import distance
+
+    distance.USE_TENSOR_CORES = bool(mma)
+    pages_per_req = -(-(context + tokens) // block_size)
+    num_pages = batch * pages_per_req + 1
+    g = torch.Generator(device="cuda").manual_seed(0)
+    pool = torch.randn((num_pages, block_size * hkv * (dk + dv)), generator=g, device="cuda").to(torch.bfloat16)
+    table = torch.randperm(num_pages - 1, generator=g, device="cuda").to(torch.int32).view(batch, pages_per_req).contiguous()
+    n = batch * tokens
+    bias = distance.DistanceBias.build(torch.randn(32, hq, device="cuda"), 1000, torch.zeros(hq, device="cuda"))
+    b = _Batch(batch, tokens, context)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    shape = dict(tokens=tokens, batch=batch, context=context, heads=hq, kv_heads=hkv, dk=dk, dv=dv, window=window, keep=keep)
+    if prep:
+        cols = hq * dk + hkv * (dk + dv)
+        proj = torch.randn(n, cols, device="cuda").to(torch.bfloat16)
+        proj_bias, first = torch.zeros(cols, device="cuda"), torch.randn(n, hkv * dv, device="cuda").to(torch.bfloat16)
+        page = table[b.token_row.long(), (b.positions // block_size).long()]
+        slots = (page * block_size + b.positions % block_size).to(torch.int32)
+        us = _time(lambda: distance.distance_prep(proj, proj_bias, 1e-5, slots, pool, hq, hkv, dk, dv, block_size,
+                                                  mix=distance.MIXED, first=first, lam=0.3), iters, flush)
+        return _result("distance_prep", us, peaks, shape, n * (2 * cols + hkv * dv) * 2)
+    q = torch.randn(n, hq * dk, device="cuda").to(torch.bfloat16)
+    fn = lambda: distance.distance_attention(q, pool, table, b.positions, b.token_row, bias, hq, hkv, dk, dv, block_size,
+                                             dk ** -0.5, window=window or None, keep_first=keep, batch=b)
+    us = _time(fn, iters, flush)
+    flops = 2.0 * (dk + dv) * hq * batch * _visible(tokens, context, window, keep)
+    keys = min(context + tokens, window + keep + tokens) if window else context + tokens
+    nbytes = batch * keys * hkv * (dk + dv) * 2 + n * hq * (dk + dv) * 2
+    return _result("distance_attention (mma.sync)" if mma else "distance_attention (CUDA cores)", us, peaks, shape, nbytes,
+                   flops)
+
+
+def depth_conv(tokens=2048, batch=1, hidden=2048, taps=4, streams=0, splits=0, iters=5, peaks=None):
+    """The kernel between two sublayers: norm and add of the sublayer's result (a tensor, or ``splits`` unsummed fp32
+    parts), the average over ``streams`` earlier streams (0: none), the convolution over time."""
+    from gllm_b200 import ops
+    from gllm_b200.ops import depth
+
+    n = tokens * batch
+    b = _Batch(batch, tokens, 0)
+    resid = torch.randn(n, hidden, device="cuda")
+    parts = torch.randn(max(splits, 1), n, hidden, device="cuda")
+    value = ops.SplitSum(parts, torch.bfloat16) if splits else parts[0].to(torch.bfloat16)
+    hist = torch.randn(streams + 1, n, hidden, device="cuda") if streams else None
+    pending = ops.DepthPending(value, None, torch.ones(hidden, device="cuda"), 1e-5, hist, streams,
+                               torch.ones(streams + 1, device="cuda") if streams else None)
+    conv_w = torch.randn(taps, hidden, device="cuda")
+    state = torch.zeros(batch + 1, taps - 1, hidden, device="cuda")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    us = _time(lambda: depth.depth_conv(pending, resid, conv_w, state, b.cu_q, b.state_slots, batch, tokens, torch.bfloat16),
+               iters, flush)
+    per = (4 * splits if splits else 2) + 4 + 4 + 2 + (4 * streams + 4 if streams else 0)
+    return _result("depth_conv", us, peaks, dict(tokens=tokens, batch=batch, hidden=hidden, taps=taps, streams=streams,
+                                                 splits=splits),
+                   n * hidden * per + batch * 2 * (taps - 1) * hidden * 4 + hidden * 4 * (taps + 1))
+
+
 KERNELS = {
+    "distance_attention": distance_attention,
+    "depth_conv": depth_conv,
     "differential_attention": differential_attention,
     "step_sized_recurrence": step_sized_recurrence,
     "add_dyt": add_dyt,

@@ -135,7 +135,7 @@ def attention(h, p, m, w, pre, eps, state, first_values):
             first_values = v
         else:
             lam = w[pre + ".vmix"].reshape(())
-            v = (1 - lam) * v + lam * first_values
+            v = (1 - lam) * v + lam * first_values.reshape(v.shape)
     state["k"], state["v"] = torch.cat([state["k"], k]), torch.cat([state["v"], v])
     S, table = state["k"].shape[0], w[pre + ".rel"]
     buckets = torch.tensor([distance_bucket(n, table.shape[0], m["bias_max"]) for n in range(S)])

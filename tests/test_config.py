@@ -131,3 +131,5 @@ def test_presets_parse():
     assert not load_config(load_preset("llama-3.1-8b")).tie_word_embeddings
     wide = load_config(load_preset("sazisun-w2048"))
     assert wide.architecture == "Sazisun" and wide.hidden_size == 2048 and wide.layers[3].mixer["kv_from"] == 1
+    wide = load_config(load_preset("vonedra-w2048"))
+    assert wide.architecture == "Vonedra" and wide.conv_taps == 4 and wide.value_mixing_layers() == [0, 3]

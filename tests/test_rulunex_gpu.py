@@ -187,7 +187,7 @@ def check_decisive(cfg, weights, runner, toks, key_at, dtype, seen=True):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("kind", ["latent", "latent_wide"])
-def test_a_far_key_at_page_and_block_edges(kind, dtype, tmp_path):
+def test_a_far_key_at_page_and_block_edges(kind, dtype, tmp_path, monkeypatch):
     from gllm_b200.engine.replay import build_runner
 
     cfg, weights = decisive_latent_model(kind)
@@ -198,6 +198,8 @@ def test_a_far_key_at_page_and_block_edges(kind, dtype, tmp_path):
     if dtype == "bfloat16":
         from gllm_b200.ops import latent
 
+        # the narrow model stays on the CUDA-core kernel, the wide one takes the tensor cores
+        monkeypatch.setattr(latent, "USE_TENSOR_CORES", kind == "latent_wide")
         m = cfg["layers"][0]["mixer"]
         assert latent.tensor_core_kernel_takes(torch.bfloat16, m["kv_rank"], m["rot_dim"]) == (kind == "latent_wide")
     for far in (0, 15, 16, 17, 31, 32, 33, 63, 64, 255, 256, 511):
