@@ -23,6 +23,11 @@
 // turn, and the first merges the two (reference maximum, sum, output) through distributed shared memory
 // at the end; the chain of tiles, which bounds a small grid, is half as long.
 //
+// BIAS: the form for attention with a learned bias by distance (attention_distance.cu has the mechanism): the table
+// of biases of the CTA's heads lies in shared memory and each score takes its own, v * scale + bias[head][distance], before
+// the softmax; with a window the first `keep_first` keys stay visible (the tiles that hold them come before the
+// window's); the sink joins the row's sum at the end.
+//
 // V is used as it lies in the cache ([key][dim], i.e. the "MN-major" operand of the second
 // product); nothing is transposed or gathered.  Keys outside a row's view get probability 0 and the
 // value rows that hold no key of the request are zeroed in shared memory before they are
@@ -129,13 +134,26 @@ struct TShape {
   static_assert(COL_P + 64 <= TMEM_COLS, "tensor memory columns");
 };
 
-template <int D>
+// What the BIAS form reads beside the rest (unused otherwise).
+struct DistanceArgs {
+  const float* bias;         // [hq][bias_len], times log2(e); every distance from bias_len - 1 on has the last value
+  int bias_len;
+  const float* sink;         // [hq] times log2(e), or null
+  int keep_first;
+  int table_ld;              // row stride of the table in shared memory, >= bias_len + 2 * BIAS_PAD
+};
+// A chunk of 32 keys reads 32 neighbouring entries of the table: it is padded by 31 on both sides so that clamping the
+// first of them is enough.
+constexpr int BIAS_PAD = 31;
+
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(THREADS, TShape<D>::CTAS_PER_SM)
 prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                     __nv_bfloat16* __restrict__ out, int64_t out_stride, const int* __restrict__ block_table,
                     int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ ctx_lens,
                     const int* __restrict__ slots, int hq, int hkv, int gp, int block_size, int num_pages,
-                    float scale_log2, int window, int* __restrict__ status, int pair, int split_min) {
+                    float scale_log2, int window, int* __restrict__ status, int pair, int split_min,
+                    const DistanceArgs dist) {
   using S = TShape<D>;
   constexpr int NB = S::NBUF;                            // score buffers in tensor memory
   constexpr int KS = S::KV_STAGES;                       // K (and V) stages in shared memory
@@ -200,12 +218,26 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   const int ctx = ctx_lens[r];
   const int pos_first = ctx + t0, pos_last = ctx + t0 + t_count - 1;
   const int kv_lo = window > 0 ? max(0, pos_first - window + 1) : 0;
-  const int tile_first = kv_lo / BN, tile_last = pos_last / BN;
-  const int n_all = has_rows ? tile_last - tile_first + 1 : 0;        // key tiles of these rows
+  const int tile_last = pos_last / BN;
+  const int keep = BIAS && window > 0 ? dist.keep_first : 0;          // keys below this one are seen beside the window
+  int tile_first = kv_lo / BN, n_kept = (keep + BN - 1) / BN;         // tiles of those keys come first
+  if (BIAS && tile_first <= n_kept && n_kept > 0) tile_first = n_kept = 0;
+  const int n_all = has_rows ? n_kept + tile_last - tile_first + 1 : 0;        // key tiles of these rows
   const int nsplit = (pair > 1 && n_all >= split_min) ? 2 : 1;        // the same in both CTAs of a pair
   const bool active = has_rows && (nsplit == 2 || rank == 0);
   const int n_tiles = active ? (n_all - (int)rank + nsplit - 1) / nsplit : 0;   // this CTA's: tile_of(0), tile_of(1), ..
-  auto tile_of = [&](int j) { return tile_first + (int)rank + nsplit * j; };
+  auto tile_of = [&](int j) {
+    const int t = (int)rank + nsplit * j;
+    return !BIAS ? tile_first + t : (t < n_kept ? t : tile_first + t - n_kept);
+  };
+  float* table = reinterpret_cast<float*>(base_ptr + S::OFF_V + KS * S::KV_STAGE);
+  if constexpr (BIAS) {
+    for (int g = 0; g < gp; ++g)
+      for (int e = threadIdx.x; e < dist.bias_len + 2 * BIAS_PAD; e += THREADS)
+        table[g * dist.table_ld + e] =
+            dist.bias[(int64_t)(h0 + g) * dist.bias_len + min(max(e - BIAS_PAD, 0), dist.bias_len - 1)];
+    __syncthreads();
+  }
 
   if (active && warp == 0) {
     // ------------------------------------------------------------------ TMA producer
@@ -224,7 +256,8 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     auto lookup = [&](int j) -> int {
       int page = -1;
       const int key = tile_of(j) * BN + lane * block_size;
-      if (j < n_tiles && lane < pages_per_tile && key <= pos_last && key + block_size > kv_lo) {
+      if (j < n_tiles && lane < pages_per_tile && key <= pos_last &&
+          (key + block_size > kv_lo || (BIAS && key < keep))) {
         page = bt[key / block_size];
         if (page >= num_pages) {
           atomicOr(status, GLLM_STATUS_PAGE_RANGE);
@@ -350,6 +383,9 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const uint32_t tmem_o = tmem_base + S::COL_O + lane_addr + (uint32_t)(hsel * HD);
     const uint32_t tmem_p = tmem_base + S::COL_P + lane_addr + (uint32_t)(hsel * HK / 2);
     float m = -INFINITY, l = 0.f;
+    // (with a bias the scores are brought to log2 units when they are read)
+    const float sl = BIAS ? 1.f : scale_log2;
+    const float* my_bias = BIAS ? table + g * dist.table_ld + BIAS_PAD : nullptr;
     bool ok = true;
     // Head size 64: one pass per tile.  The probabilities are taken against the reference maximum the row
     // already has while the tile's maximum is found on the side; only when some row's maximum has outgrown
@@ -375,8 +411,8 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 #pragma unroll
       for (int ci = 0; ci < HK / 32; ++ci) {
         const int k0 = kv0 + ci * 32;
-        const bool none = k0 > pos_last || k0 + 31 < kv_lo;
-        const bool all = k0 + 31 <= pos_first && (window <= 0 || k0 >= pos_last - window + 1);
+        const bool none = k0 > pos_last || (k0 + 31 < kv_lo && (!BIAS || k0 >= keep));
+        const bool all = k0 + 31 <= pos_first && (window <= 0 || k0 >= pos_last - window + 1 || (BIAS && k0 + 31 < keep));
         cls[ci] = none ? CHUNK_SKIP : all ? CHUNK_FAST : CHUNK_MASK;
       }
       // the tile's scores -> (maximum) and/or (probabilities in tensor memory, their sums)
@@ -394,9 +430,30 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 #pragma unroll
         for (int ci = 0; ci < HK / 32; ++ci) {
           uint32_t packed[16];
-          if (cls[ci] == CHUNK_FAST) {
-            softmax_chunk<false, WM, WE>(v[ci], 0, 0u, scale_log2, neg_mc, mx, lsum, packed);
-          } else if (cls[ci] == CHUNK_MASK) {
+          if constexpr (BIAS) {
+            if (cls[ci] != CHUNK_SKIP) {
+              const int k0 = kv0 + ci * 32;
+              const float* b = my_bias + min(max(qpos - k0, 0), dist.bias_len - 1 + BIAS_PAD);
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                const float2 t = ffma2(make_float2(v[ci][i], v[ci][i + 1]), make_float2(scale_log2, scale_log2),
+                                       make_float2(b[-i], b[-i - 1]));
+                v[ci][i] = t.x;
+                v[ci][i + 1] = t.y;
+              }
+              // hidden keys: the general mask below knows one stretch of keys, the kept ones are a second
+              if (cls[ci] == CHUNK_MASK) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) {
+                  const int key = k0 + i;
+                  if (!(key <= hi && (key >= lo || key < keep))) v[ci][i] = -INFINITY;
+                }
+              }
+            }
+          }
+          if (cls[ci] == CHUNK_FAST || (BIAS && cls[ci] == CHUNK_MASK)) {
+            softmax_chunk<false, WM, WE>(v[ci], 0, 0u, sl, neg_mc, mx, lsum, packed);
+          } else if (!BIAS && cls[ci] == CHUNK_MASK) {
             softmax_chunk<true, WM, WE>(v[ci], kv0 + ci * 32 - lo_eff, span, scale_log2, neg_mc, mx, lsum, packed);
           } else {
 #pragma unroll
@@ -418,7 +475,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       float mx = -INFINITY;
       float2 lsum = make_float2(0.f, 0.f);
       if (speculate) {
-        pass(Yes{}, Yes{}, true, -(m == -INFINITY ? 0.f : m) * scale_log2, mx, lsum);
+        pass(Yes{}, Yes{}, true, -(m == -INFINITY ? 0.f : m) * sl, mx, lsum);
       } else {
         pass(Yes{}, No{}, false, 0.f, mx, lsum);
       }
@@ -434,11 +491,11 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       // exponent: until then the exponentials are taken against the old one (they stay below 256, exact
       // enough in fp32 and bf16, and the final division by the row's sum takes the common factor out),
       // and the output so far needs no rescaling, which is the usual case after a row's first tiles.
-      const bool moves = mx > -INFINITY && (m == -INFINITY || (mx - m) * scale_log2 > 8.0f);
+      const bool moves = mx > -INFINITY && (m == -INFINITY || (mx - m) * sl > 8.0f);
       const float m_new = moves ? fmaxf(m, mx) : m;
       if (!speculate || __any_sync(0xffffffffu, moves)) {
         const float m_use = m_new == -INFINITY ? 0.f : m_new;
-        const float corr = m == -INFINITY ? 0.f : fast_exp2((m - m_use) * scale_log2);
+        const float corr = m == -INFINITY ? 0.f : fast_exp2((m - m_use) * sl);
         // the output so far is rescaled when some row of the warp saw its maximum move
         if (j > 0) {
           if (!speculate) {
@@ -459,7 +516,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         l *= corr;
         lsum = make_float2(0.f, 0.f);
         float unused = 0.f;
-        pass(No{}, Yes{}, false, -m_use * scale_log2, unused, lsum);
+        pass(No{}, Yes{}, false, -m_use * sl, unused, lsum);
         tmem_wait_st();
       }
       m = m_new;
@@ -470,7 +527,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (tile0 + BN - 1 > pos_last || tile0 < kv_lo) {
         mbar_wait(smem_addr(&v_full[j % KS]), (uint32_t)(j / KS) & 1u, status, &abort_flag);
         const int key = tile0 + row;                     // thread <-> key row of the V tile (lower-half warps)
-        if (hsel == 0 && (key > pos_last || key < kv_lo)) {
+        if (hsel == 0 && (key > pos_last || (key < kv_lo && (!BIAS || key >= keep)))) {
           for (int db = 0; db < S::DB; ++db) {
             uint4* vrow =
                 reinterpret_cast<uint4*>(base_ptr + S::OFF_V + (j % KS) * S::KV_STAGE + db * S::TILE + row * 128);
@@ -490,6 +547,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     asm volatile("bar.sync 1, 256;" ::: "memory");
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const float l_row = l + row_max[hsel ^ 1][row];
+    const float sink = BIAS && dist.sink != nullptr ? dist.sink[h0 + g] : -INFINITY;
     __nv_bfloat16* dst = out + (int64_t)(tok_begin + t0 + tl) * out_stride + (int64_t)(h0 + g) * D + hsel * HD;
     auto store32 = [&](int c, const float (&v)[32], float inv) {
       if (row_ok) {
@@ -505,7 +563,8 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     };
     if (nsplit == 1) {
       if (ok && n_tiles > 0 && !abort_flag) {
-        const float inv = l_row > 0.f ? 1.0f / l_row : 0.f;
+        const float l_all = BIAS ? l_row + fast_exp2(sink - (m == -INFINITY ? sink : m)) : l_row;
+        const float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
 #pragma unroll 1
         for (int c = 0; c < HD; c += 32) {
           float v[32];
@@ -550,9 +609,10 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(l1) : "r"(r_l) : "memory");
         // (this CTA has a tile whenever the rows have one; a row that saw nothing keeps m = -inf, l = 0)
         const float mm = fmaxf(m, m1);
-        const float a0 = m == -INFINITY ? 0.f : fast_exp2((m - mm) * scale_log2);
-        const float a1 = m1 == -INFINITY ? 0.f : fast_exp2((m1 - mm) * scale_log2);
-        const float l_all = a0 * l_row + a1 * l1;
+        const float a0 = m == -INFINITY ? 0.f : fast_exp2((m - mm) * sl);
+        const float a1 = m1 == -INFINITY ? 0.f : fast_exp2((m1 - mm) * sl);
+        float l_all = a0 * l_row + a1 * l1;
+        if (BIAS && mm > -INFINITY) l_all += fast_exp2(sink - mm);
         const float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
         const bool good = ok && !abort_flag;
 #pragma unroll 1
@@ -605,12 +665,12 @@ EncodeTiledFn encode_fn() {
   return fn;
 }
 
-template <int D>
+template <int D, bool BIAS>
 int prefill_tmem_launch(const __nv_bfloat16* q, int64_t q_stride, __nv_bfloat16* out, int64_t out_stride,
                         const __nv_bfloat16* cache, const int* block_table, int bt_stride, const int* cu_q,
                         const int* ctx_lens, const int* slots, int num_requests, int max_q_len, int n_tokens,
                         int hq, int hkv, int block_size, int num_pages, float scale, int window, int* status,
-                        cudaStream_t stream) {
+                        cudaStream_t stream, DistanceArgs dist = {}) {
   using S = TShape<D>;
   EncodeTiledFn fn = encode_fn();
   if (!fn) return (int)cudaErrorNotSupported;
@@ -640,11 +700,13 @@ int prefill_tmem_launch(const __nv_bfloat16* q, int64_t q_stride, __nv_bfloat16*
            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
       return (int)cudaErrorInvalidValue;
   }
-  static bool attr_set = false;
-  if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_tmem_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::SMEM);
+  const size_t smem = (size_t)S::SMEM + (BIAS ? sizeof(float) * (size_t)gp * dist.table_ld : 0);
+  static size_t smem_set = 0;
+  if (smem > smem_set) {
+    cudaError_t e =
+        cudaFuncSetAttribute(prefill_tmem_kernel<D, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    attr_set = true;
+    smem_set = smem;
   }
   dim3 grid(hkv * (group / gp), (max_q_len + qt - 1) / qt, num_requests);
   // A small grid is bound by its longest CTA's chain of key tiles, not by the SMs' throughput.  Where twice the grid
@@ -662,13 +724,13 @@ int prefill_tmem_launch(const __nv_bfloat16* q, int64_t q_stride, __nv_bfloat16*
   const int64_t places = (int64_t)gllm_sm_count() * S::CTAS_PER_SM;
   if (pair_on && 2 * (int64_t)grid.x * grid.y * grid.z <= places) {
     grid.x *= 2;
-    return gllm_launch_cluster(prefill_tmem_kernel<D>, grid, dim3(THREADS), (size_t)S::SMEM, stream, 2u, map_q, map_kv, out,
+    return gllm_launch_cluster(prefill_tmem_kernel<D, BIAS>, grid, dim3(THREADS), smem, stream, 2u, map_q, map_kv, out,
                                out_stride, block_table, bt_stride, cu_q, ctx_lens, slots, hq, hkv, gp, block_size,
-                               num_pages, scale * 1.4426950408889634f, window, status, 2, split_min);
+                               num_pages, scale * 1.4426950408889634f, window, status, 2, split_min, dist);
   }
-  return gllm_launch(prefill_tmem_kernel<D>, grid, dim3(THREADS), (size_t)S::SMEM, stream, map_q, map_kv, out,
+  return gllm_launch(prefill_tmem_kernel<D, BIAS>, grid, dim3(THREADS), smem, stream, map_q, map_kv, out,
                      out_stride, block_table, bt_stride, cu_q, ctx_lens, slots, hq, hkv, gp, block_size, num_pages,
-                     scale * 1.4426950408889634f, window, status, 1, split_min);
+                     scale * 1.4426950408889634f, window, status, 1, split_min, dist);
 }
 }  // namespace
 
@@ -691,10 +753,48 @@ GLLM_API int gllm_attention_prefill_tmem(const __nv_bfloat16* q, int64_t q_strid
       (reinterpret_cast<uintptr_t>(cache) & 15) || (reinterpret_cast<uintptr_t>(out) & 15) || num_pages < 1)
     return (int)cudaErrorInvalidValue;
   if (d == 64)
-    return prefill_tmem_launch<64>(q, q_stride, out, out_stride, cache, block_table, bt_stride, cu_q, ctx_lens, slots,
+    return prefill_tmem_launch<64, false>(q, q_stride, out, out_stride, cache, block_table, bt_stride, cu_q, ctx_lens, slots,
                                    num_requests, max_q_len, n_tokens, hq, hkv, block_size, num_pages, scale, window,
                                    status, stream);
-  return prefill_tmem_launch<128>(q, q_stride, out, out_stride, cache, block_table, bt_stride, cu_q, ctx_lens, slots,
+  return prefill_tmem_launch<128, false>(q, q_stride, out, out_stride, cache, block_table, bt_stride, cu_q, ctx_lens, slots,
                                   num_requests, max_q_len, n_tokens, hq, hkv, block_size, num_pages, scale, window,
                                   status, stream);
+}
+
+// Row stride of the BIAS form's table in shared memory (the heads of a warp's rows read different banks).
+static int distance_table_ld(int gp, int bias_len) {
+  const int odd = gp >= 32 ? 1 : 32 / gp;
+  return (bias_len + 2 * BIAS_PAD - odd + 31) / 32 * 32 + odd;
+}
+
+// 1 when the BIAS form takes these sizes (keys and values of one width, a table that fits beside the tiles).
+GLLM_API int gllm_attention_prefill_distance_supports(int hq, int hkv, int d, int block_size, int bias_len) {
+  if (!gllm_attention_prefill_tmem_supports(d, block_size) || hq <= 0 || hkv <= 0 || hq % hkv || bias_len < 1) return 0;
+  const int group = hq / hkv, gp = (group <= BM && BM % group == 0) ? group : 1;
+  const size_t table = sizeof(float) * (size_t)gp * distance_table_ld(gp, bias_len);
+  return table + (d == 64 ? TShape<64>::SMEM : TShape<128>::SMEM) <= 220 * 1024 ? 1 : 0;
+}
+
+// As gllm_attention_prefill_tmem with a bias by distance, kept first tokens and a sink (bias and sink times log2(e)).
+GLLM_API int gllm_attention_prefill_distance(const __nv_bfloat16* q, int64_t q_stride, __nv_bfloat16* out,
+                                             int64_t out_stride, const __nv_bfloat16* cache, const int* block_table,
+                                             int bt_stride, const int* cu_q, const int* ctx_lens, const int* slots,
+                                             const float* bias, int bias_len, const float* sink, int num_requests,
+                                             int max_q_len, int n_tokens, int hq, int hkv, int d, int block_size,
+                                             int num_pages, float scale, int window, int keep_first, int* status,
+                                             cudaStream_t stream) {
+  if (num_requests <= 0 || max_q_len <= 0) return 0;
+  if (!gllm_attention_prefill_distance_supports(hq, hkv, d, block_size, bias_len) || bias == nullptr || window < 0 ||
+      keep_first < 0 || num_requests > 65535 || (q_stride % 8) || (out_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15) ||
+      (reinterpret_cast<uintptr_t>(cache) & 15) || (reinterpret_cast<uintptr_t>(out) & 15) || num_pages < 1)
+    return (int)cudaErrorInvalidValue;
+  const int group = hq / hkv, gp = (group <= BM && BM % group == 0) ? group : 1;
+  const DistanceArgs dist{bias, bias_len, sink, keep_first, distance_table_ld(gp, bias_len)};
+  if (d == 64)
+    return prefill_tmem_launch<64, true>(q, q_stride, out, out_stride, cache, block_table, bt_stride, cu_q, ctx_lens, slots,
+                                         num_requests, max_q_len, n_tokens, hq, hkv, block_size, num_pages, scale, window,
+                                         status, stream, dist);
+  return prefill_tmem_launch<128, true>(q, q_stride, out, out_stride, cache, block_table, bt_stride, cu_q, ctx_lens, slots,
+                                        num_requests, max_q_len, n_tokens, hq, hkv, block_size, num_pages, scale, window,
+                                        status, stream, dist);
 }

@@ -1,5 +1,6 @@
-"""Python entry points of ``csrc/attention_distance.cu`` and ``csrc/attention_distance_mma.cu``: softmax attention with
-a learned bias by distance, a window that keeps the first tokens, and a sink.  As everywhere in ``gllm_b200.ops``: CUDA
+"""Python entry points of ``csrc/attention_distance.cu`` and ``csrc/attention_distance_mma.cu`` (and of the form with a
+bias of ``csrc/attention_prefill_tmem.cu``): softmax attention with a learned bias by distance, a window that keeps the
+first tokens, and a sink.  As everywhere in ``gllm_b200.ops``: CUDA
 tensors only, no CPU path."""
 
 from __future__ import annotations
@@ -16,9 +17,13 @@ from gllm_b200.ops import _check, _cuda, _fn, _parts_args, _ptr, _stream, _suffi
 
 # GLLM_B200_DISTANCE_MMA=0: the attention of bf16 models stays on the CUDA-core kernel (for measurements)
 USE_TENSOR_CORES = os.environ.get("GLLM_B200_DISTANCE_MMA", "1") != "0"
-KEY_TILE = 64
-SPLIT_TILES = 2           # key tiles per CTA at least when single tokens' contexts are cut
+KEY_TILE = 64             # keys of a tile of portions, and of single tokens
+SINGLE_KEY_TILE = 32
+SPLIT_TILES = 2           # key tiles per CTA at least when the keys of short portions are cut, and of single tokens
+SINGLE_SPLIT_TILES = 4
 MAX_SPLITS = 16
+# portions shorter than this stay on the mma.sync kernel (its 64-row tiles waste less on short portions)
+TMEM_MIN_Q_LEN = 32
 
 NO_MIX, FIRST, MIXED = 0, 1, 2        # what the prep kernel does with the values
 
@@ -35,11 +40,39 @@ def _mma_fns():
         lib = load_module("attention_distance_mma")
         f = lib.gllm_attention_distance_mma
         f.argtypes = [P, c_int64, P, c_int64, P, P, c_int, P, P, c_int, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
-                      c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, P, P]
+                      c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, P, P]
         f.restype = c_int
         lib.gllm_attention_distance_mma_tokens_per_tile.argtypes = [c_int, c_int]
-        _mma = (f, lib.gllm_attention_distance_mma_tokens_per_tile)
+        lib.gllm_attention_distance_few_tiles.argtypes = [c_int, c_int]
+        _mma = (f, lib.gllm_attention_distance_mma_tokens_per_tile, lib.gllm_attention_distance_few_tiles)
     return _mma
+
+
+_tmem = None
+
+
+def _tmem_fns():
+    global _tmem
+    if _tmem is None:
+        from ctypes import c_float, c_int, c_int64, c_void_p as P
+
+        from gllm_b200.ops.build import load_module
+
+        lib = load_module("attention_prefill_tmem")
+        f = lib.gllm_attention_prefill_distance
+        f.argtypes = [P, c_int64, P, c_int64, P, P, c_int, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int,
+                      c_int, c_int, c_float, c_int, c_int, P, P]
+        f.restype = c_int
+        lib.gllm_attention_prefill_distance_supports.argtypes = [c_int, c_int, c_int, c_int, c_int]
+        _tmem = (f, lib.gllm_attention_prefill_distance_supports)
+    return _tmem
+
+
+def takes_tmem(heads: int, kv_heads: int, dk: int, dv: int, block_size: int, bias_len: int) -> bool:
+    """True for the sizes the tcgen05 kernel takes: keys and values both 64 or both 128 wide, pages of a power of two
+    of tokens, a bias table that fits shared memory."""
+    return (dk == dv and dk in (64, 128)
+            and bool(_tmem_fns()[1](heads, kv_heads, dk, block_size, bias_len)))
 
 
 def takes_tensor_cores(dtype: torch.dtype, dk: int, dv: int) -> bool:
@@ -134,23 +167,49 @@ def distance_prep(proj, bias: torch.Tensor | None, eps: float, slot_mapping: tor
     return q
 
 
-def _splits(batch, n_rows_tile: int, head_tiles: int, window: int, keep_first: int, table_tokens: int, device):
-    """(ranges, key tiles per range) of a step: one range unless its tiles do not fill the GPU."""
-    # a captured prompt portion is replayed for other contexts: under capture the ranges cover what a block-table
-    # row can hold, not just the captured step's longest sequence (single tokens are captured per sequence bucket)
-    longest = batch.max_seq_len
-    if batch.max_q_len > 1 and torch.cuda.is_current_stream_capturing():
-        longest = max(longest, table_tokens)
-    most = -(-longest // KEY_TILE)
-    if window:
-        most = min(most, -(-keep_first // KEY_TILE) + -(-(window + n_rows_tile) // KEY_TILE) + 1)
-    tiles = -(-batch.max_q_len // n_rows_tile) * head_tiles * batch.num_requests
+def _ranges(most: int, tiles: int, least: int, per_sm: int, device):
+    """(ranges, key tiles per range) for CTAs that visit up to ``most`` key tiles, ``tiles`` of them in all: one range
+    unless they do not fill the GPU."""
     sms = torch.cuda.get_device_properties(device).multi_processor_count
-    if 2 * tiles > sms or most < 2 * SPLIT_TILES:
+    if 2 * tiles > sms * per_sm or most < 2 * least:
         return 1, 0
-    want = min(MAX_SPLITS, -(-4 * sms // tiles))
-    per = max(SPLIT_TILES, -(-most // want))
+    want = min(MAX_SPLITS, -(-per_sm * sms // tiles))
+    per = max(least, -(-most // want))
     return -(-most // per), per
+
+
+def _visited(longest: int, tile: int, tokens: int, window: int, keep_first: int) -> int:
+    """The most key tiles that ``tokens`` neighbouring tokens visit."""
+    most = -(-longest // tile)
+    return min(most, -(-keep_first // tile) + -(-(window + tokens) // tile) + 1) if window else most
+
+
+def _mma_launch(q, out, pages, block_table, bias, heads, kv_heads, dk, dv, block_size, scale, window, keep_first, batch,
+                first: int, count: int, single: bool):
+    """The mma.sync kernels over requests ``first .. first+count-1`` (``single``: each brings one token)."""
+    f, tokens_per_tile, few_tiles = _mma_fns()
+    n, longest = q.shape[0], batch.max_seq_len
+    if single:
+        splits, per = _ranges(_visited(longest, SINGLE_KEY_TILE, 1, window, keep_first), few_tiles(heads, kv_heads) * count,
+                              SINGLE_SPLIT_TILES, 2, q.device)
+    else:
+        # a captured prompt portion is replayed for other contexts: under capture the ranges cover what a block-table
+        # row can hold, not just the captured step's longest sequence (single tokens are captured per sequence bucket)
+        if torch.cuda.is_current_stream_capturing():
+            longest = max(longest, block_table.shape[1] * block_size)
+        qt = tokens_per_tile(heads, kv_heads)
+        splits, per = _ranges(_visited(longest, KEY_TILE, qt, window, keep_first),
+                              -(-batch.max_q_len // qt) * (heads * qt // 64) * count, SPLIT_TILES, 2, q.device)
+    partial = stats = None
+    if splits > 1:
+        partial = batch.workspace.get("distance_attention_partial", splits * n * heads * dv, torch.float32)
+        stats = batch.workspace.get("distance_attention_stats", splits * n * heads * 2, torch.float32)
+    _check(f(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), _ptr(partial), _ptr(stats), n, pages.data_ptr(),
+             block_table.data_ptr(), block_table.stride(0), batch.cu_q[first:].data_ptr(),
+             batch.context_lens[first:].data_ptr(), batch.state_slots[first:].data_ptr(), bias.table_log2.data_ptr(),
+             bias.table_log2.shape[1], _ptr(bias.sink_log2), count, 1 if single else batch.max_q_len, heads, kv_heads, dk,
+             dv, int(block_size), pages.shape[0], float(scale), window, keep_first, int(single), splits, per,
+             status_word(q.device).data_ptr(), _stream()), "distance_attention_mma")
 
 
 def distance_attention(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor,
@@ -175,19 +234,23 @@ def distance_attention(q: torch.Tensor, pages: torch.Tensor, block_table: torch.
     out = torch.empty((n, heads * dv), dtype=q.dtype, device=q.device)
     if (batch is not None and USE_TENSOR_CORES and takes_tensor_cores(q.dtype, dk, dv) and q.stride(0) % 8 == 0
             and q.data_ptr() % 16 == 0):
-        f, tokens_per_tile = _mma_fns()
-        qt = tokens_per_tile(heads, kv_heads)
-        splits, per = _splits(batch, qt, heads * qt // KEY_TILE, win, int(keep_first), block_table.shape[1] * block_size, q.device)
-        partial = stats = None
-        if splits > 1:
-            partial = batch.workspace.get("distance_attention_partial", splits * n * heads * dv, torch.float32)
-            stats = batch.workspace.get("distance_attention_stats", splits * n * heads * 2, torch.float32)
-        code = f(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), _ptr(partial), _ptr(stats), n, pages.data_ptr(),
-                 block_table.data_ptr(), block_table.stride(0), batch.cu_q.data_ptr(), batch.context_lens.data_ptr(),
-                 batch.state_slots.data_ptr(), bias.table_log2.data_ptr(), bias.table_log2.shape[1], _ptr(bias.sink_log2),
-                 batch.num_requests, batch.max_q_len, heads, kv_heads, dk, dv, int(block_size), pages.shape[0],
-                 float(scale), win, int(keep_first), splits, per, status_word(q.device).data_ptr(), _stream())
-        _check(code, "distance_attention_mma")
+        # the flat batch holds the portions first, then the single tokens: each kind has a kernel of its own
+        portions = getattr(batch, "num_prefill_requests", None)
+        if portions is None:
+            portions = 0 if batch.max_q_len == 1 else batch.num_requests
+        args = (bias, heads, kv_heads, dk, dv, block_size, scale, win, int(keep_first), batch)
+        if portions and batch.max_q_len >= TMEM_MIN_Q_LEN and takes_tmem(heads, kv_heads, dk, dv, block_size,
+                                                                        bias.table.shape[1]):
+            _check(_tmem_fns()[0](q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), pages.data_ptr(),
+                                  block_table.data_ptr(), block_table.stride(0), batch.cu_q.data_ptr(),
+                                  batch.context_lens.data_ptr(), batch.state_slots.data_ptr(), bias.table_log2.data_ptr(),
+                                  bias.table_log2.shape[1], _ptr(bias.sink_log2), portions, batch.max_q_len, n, heads,
+                                  kv_heads, dk, int(block_size), pages.shape[0], float(scale), win, int(keep_first),
+                                  status_word(q.device).data_ptr(), _stream()), "distance_attention_tmem")
+        elif portions:
+            _mma_launch(q, out, pages, block_table, *args, 0, portions, False)
+        if portions < batch.num_requests:
+            _mma_launch(q, out, pages, block_table, *args, portions, batch.num_requests - portions, True)
         return out
     f = _fn("attention_distance", f"gllm_attention_distance_{_suffix(q.dtype)}")
     _check(f(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), pages.data_ptr(), block_table.data_ptr(),

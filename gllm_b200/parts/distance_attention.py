@@ -50,7 +50,9 @@ class DistanceAttention(Mixer):
         self.lam = 0.0
 
     def kernel_needs(self):
-        return {"modules": {"attention_distance", "attention_distance_mma"}}
+        # the second holds the tensor-core kernels of bfloat16 runs, the third the one for longer portions
+        wide = {"attention_prefill_tmem"} if self.dk == self.dv and self.dk in (64, 128) else set()
+        return {"modules": {"attention_distance", "attention_distance_mma"} | wide}
 
     def kv_requirement(self):
         return KVPageRequirement(((self.kv_heads, self.dk), (self.kv_heads, self.dv)), self.window, self.keep_first)

@@ -18,6 +18,9 @@ from tiny_vonedra import VONEDRA, _att, _delta, _latent, draw_weights, one_layer
 pytestmark = pytest.mark.gpu
 
 PAGE = {"A": 4, "B": 8, "C": 16, "D": 32}
+# seeds of the weights: models whose logits rounding alone does not move by several per cent (a result that is nearly
+# zero before its norm does that)
+SEED = {"A": 7, "B": 7, "C": 8, "D": 7}
 F = plain.F
 
 
@@ -62,6 +65,8 @@ class Step:
         self.positions = torch.cat([torch.arange(s, s + n) for s, n in zip(starts, lengths)]).to(torch.int32).to(dev)
         self.token_row = torch.cat([torch.full((n,), s) for s, n in zip(slots, lengths)]).to(torch.int32).to(dev)
         self.num_requests, self.max_q_len = len(lengths), max(lengths)
+        self.num_prefill_requests = sum(n > 1 for n in lengths)
+        assert all(a >= b or b > 1 for a, b in zip(lengths, lengths[1:]))          # portions before single tokens
         self.max_seq_len = max(s + n for s, n in zip(starts, lengths))
         self.workspace = Workspace(dev)
 
@@ -182,7 +187,7 @@ def test_result_norm_depth_average_and_convolution(dtype, width, taps, streams, 
     assert taps == 1 or (float(state[0].min()) == 7.0 and float(state[5].max()) == 7.0)       # others' slots
 
 
-PLANS = [[(0, 37), (1, 9)], [(1, 1), (0, 2)], [(0, 1), (1, 1)], [(0, 64), (1, 30)], [(0, 46)]]
+PLANS = [[(0, 37), (1, 9)], [(0, 2), (1, 1)], [(0, 1), (1, 1)], [(0, 64), (1, 30)], [(0, 46)]]
 
 
 @pytest.mark.parametrize("cores", ["cuda", "tensor"])
@@ -271,7 +276,9 @@ def test_single_tokens_over_ranges_of_keys():
             st = req.step(plan)
             q = distance.distance_prep(req.rows(proj, plan).contiguous(), None, 1e-5, req.slot_map(plan), cache, heads,
                                        kv_heads, dim, vdim, page)
-            split += distance._splits(st, 32, heads // 2, size or 0, keep, req.table.shape[1] * page, q.device)[0] > 1
+            if st.max_q_len == 1:
+                most = distance._visited(st.max_seq_len, distance.SINGLE_KEY_TILE, 1, size or 0, keep)
+                split += distance._ranges(most, kv_heads * 3, distance.SINGLE_SPLIT_TILES, 2, q.device)[0] > 1
             req.take(distance.distance_attention(q, cache, req.table.cuda(), st.positions, st.token_row, table, heads,
                                                  kv_heads, dim, vdim, page, scale, window=size, keep_first=keep,
                                                  batch=st), plan)
@@ -411,8 +418,8 @@ def test_delta_rule_with_one_decay_per_head(heads, kv_heads, dim, vdim, taps):
     for s in req.slot_of.values():
         state[s] = 0
         conv_state[s] = 0
-    plans = [[(0, 7), (1, 2)], [(1, 1), (0, 2)], [(0, 1), (1, 1)], [(0, 2), (1, 1)]] if big else \
-        [[(0, 23), (1, 8)], [(1, 1), (0, 2)], [(0, 1), (1, 1)], [(0, 19), (1, 10)]]
+    plans = [[(0, 7), (1, 2)], [(0, 2), (1, 1)], [(0, 1), (1, 1)], [(0, 2), (1, 1)]] if big else \
+        [[(0, 23), (1, 8)], [(0, 2), (1, 1)], [(0, 1), (1, 1)], [(0, 19), (1, 10)]]
     for plan in plans:
         st = req.step(plan)
         raw = req.rows(ba, plan)
@@ -493,7 +500,7 @@ def test_all_cuts_and_mixed_batches(name, dtype, tmp_path):
 
     cfg = VONEDRA[name]
     weights, folder, runner = make(cfg, tmp_path, dtype, max_tokens=rounded(max(LENGTHS.values())),
-                                   block_size=PAGE[name])
+                                   block_size=PAGE[name], seed=SEED[name])
     seqs = sequences(cfg["vocab"], seed=5)
     want = {k: plain.forward(cfg, weights, v) for k, v in seqs.items()}
     steps, index = single_request_steps(seqs)
@@ -602,7 +609,7 @@ def test_portions_at_every_edge(dtype, tmp_path):
     """Portions that end one token before, at and after every page border, window edge and the end of the kept tokens,
     down to two tokens."""
     cfg = VONEDRA["C"]
-    weights, _, runner = make(cfg, tmp_path, dtype, max_tokens=256, block_size=16)
+    weights, _, runner = make(cfg, tmp_path, dtype, max_tokens=256, block_size=16, seed=SEED["C"])
     toks = torch.randint(0, cfg["vocab"], (130,), generator=torch.Generator().manual_seed(10)).tolist()
     want = {"r": plain.forward(cfg, weights, toks)}
     for cuts in ([15, 2, 15, 1, 31, 2, 34, 30], [16, 16, 1, 31, 33, 33], [36, 2, 12, 2, 17, 2, 59], [49, 2, 2, 45, 2, 2, 28],
