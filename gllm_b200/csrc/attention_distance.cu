@@ -86,6 +86,74 @@ distance_prep_kernel(const T* __restrict__ proj, int64_t stride, const float* __
   }
 }
 
+// The same for projections that arrive as a tensor, sixteen bytes a lane: `lanes` (a power of two, lanes * VEC >= both
+// widths, widths multiples of VEC) neighbouring lanes share a head, so a warp takes 32 / lanes of them.
+template <typename T>
+__global__ void __launch_bounds__(256)
+distance_prep_vec_kernel(const T* __restrict__ proj, int64_t stride, const float* __restrict__ bias, float eps,
+                         T* __restrict__ q_out, T* __restrict__ first, int mode, float lambda,
+                         const int* __restrict__ slot_mapping, T* __restrict__ cache, int n_tokens, int hq, int hkv,
+                         int dk, int dv, int lanes, int block_size, int num_pages, int* __restrict__ status) {
+  constexpr int VEC = 16 / sizeof(T);
+  pdl_trigger();
+  pdl_wait();
+  const int sub = threadIdx.x & (lanes - 1);
+  const int per_token = hq + 2 * hkv;
+  const int64_t item = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
+  const bool live = item < (int64_t)n_tokens * per_token;          // (every lane takes part in the shuffles)
+  const int n = live ? (int)(item / per_token) : 0, u = live ? (int)(item - (int64_t)n * per_token) : 0;
+  const bool is_v = u >= hq + hkv;
+  const int width = is_v ? dv : dk, c = sub * VEC;
+  const int col = is_v ? (hq + hkv) * dk + (u - hq - hkv) * dv : u * dk;
+  const bool mine = live && c < width;
+  float x[VEC], ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) x[e] = 0.f;
+  if (mine) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(proj + (int64_t)n * stride + col + c);
+    const T* r = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      x[e] = to_float(r[e]);
+      if (bias) x[e] += bias[col + c + e];
+      ss = fmaf(x[e], x[e], ss);
+    }
+  }
+  for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!mine) return;
+  if (!is_v) {
+    const float inv = 1.0f / sqrtf(ss / (float)dk + eps);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[e] *= inv;
+  } else if (mode == 2) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(first + (int64_t)n * hkv * dv + (u - hq - hkv) * dv + c);
+    const T* f = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[e] = (1.0f - lambda) * x[e] + lambda * to_float(f[e]);
+  }
+  uint4 packed;
+  T* y = reinterpret_cast<T*>(&packed);
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) y[e] = from_float<T>(x[e]);
+  if (is_v && mode == 1) *reinterpret_cast<uint4*>(first + (int64_t)n * hkv * dv + (u - hq - hkv) * dv + c) = packed;
+  T* dst;
+  if (u < hq) {
+    dst = q_out + (int64_t)n * hq * dk + (int64_t)u * dk;
+  } else {
+    const int slot = slot_mapping ? slot_mapping[n] : -1;
+    if (slot < 0) return;
+    const int page = slot / block_size, off = slot % block_size;
+    if (page >= num_pages) {
+      if (sub == 0) atomicOr(status, GLLM_STATUS_PAGE_RANGE);
+      return;
+    }
+    T* base = cache + (size_t)page * hkv * block_size * (dk + dv);
+    dst = is_v ? base + (size_t)hkv * block_size * dk + ((size_t)(u - hq - hkv) * block_size + off) * dv
+               : base + ((size_t)(u - hq) * block_size + off) * dk;
+  }
+  *reinterpret_cast<uint4*>(dst + c) = packed;
+}
+
 // One warp per (token, query head).
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
@@ -174,6 +242,18 @@ int distance_prep_launch(const T* proj, int64_t stride, const float* parts, int 
       (proj == nullptr) == (parts == nullptr) || (mode != 0 && first == nullptr) ||
       (slot_mapping != nullptr && (block_size <= 0 || cache == nullptr)))
     return (int)cudaErrorInvalidValue;
+  constexpr int VEC = 16 / (int)sizeof(T);
+  auto odd = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) != 0; };
+  if (parts == nullptr && dk % VEC == 0 && dv % VEC == 0 && dk <= 32 * VEC && dv <= 32 * VEC && stride % VEC == 0 &&
+      !odd(proj) && !odd(q_out) && !odd(first) && !odd(cache)) {
+    int lanes = 1;
+    while (lanes * VEC < dk || lanes * VEC < dv) lanes *= 2;
+    const int64_t grid = ((int64_t)n_tokens * (hq + 2 * hkv) * lanes + 255) / 256;
+    if (grid > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
+    return gllm_launch(distance_prep_vec_kernel<T>, dim3((unsigned)grid), dim3(256), 0, stream, proj, stride, bias, eps,
+                       q_out, first, mode, lambda, slot_mapping, cache, n_tokens, hq, hkv, dk, dv, lanes, block_size,
+                       num_pages, status);
+  }
   const int64_t blocks = ((int64_t)n_tokens * (hq + 2 * hkv) + WARPS - 1) / WARPS;
   if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
   return gllm_launch(distance_prep_kernel<T>, dim3((unsigned)blocks), dim3(WARPS * 32), 0, stream, proj, stride, parts,

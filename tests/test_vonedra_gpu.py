@@ -315,7 +315,8 @@ def test_values_of_the_first_layer_are_kept():
         assert torch.equal(first, v)
         want = whole.double()[:, 64:] + bias.double()[64:]
         assert torch.allclose(first.double().cpu(), want, atol=0.03, rtol=5e-3)
-    assert all(torch.equal(a, b) for a, b in zip(*results))
+    for a, b in zip(*results):                                   # (one sums a head's squares in another order)
+        assert torch.allclose(a.float(), b.float(), atol=1e-3, rtol=1e-2)
 
 
 @pytest.mark.parametrize("cores", ["cuda", "tensor"])
