@@ -3,7 +3,7 @@
 // with everything but the projections in fp32.  Three kernels:
 //   delta_prep         per token: the short causal convolution + SiLU of the q, k and v projections (over the
 //                      request's own earlier tokens and its convolution state), q and k made unit vectors per head
-//                      (q also times q_scale), the decays g = exp(-exp(A_log[h]) softplus(a + dt_bias)) and
+//                      (q also times q_scale), the decays' losses 1 - g, g = exp(-exp(A_log[h]) softplus(a + dt_bias)) and
 //                      beta = sigmoid(b);
 //   conv_state_update  per request: the last taps-1 inputs of the convolution become its new state;
 //   delta_rule         per (request, head, block of value columns): the recurrence, token after token.
@@ -13,6 +13,8 @@
 // one round of shuffles per token instead of two.  The state is stored column by column, [slots, heads, dv, dk],
 // as the other matrix recurrences store theirs.
 // The decays come per key channel, g [n, heads * dk], or one per head, g [n, heads] (`decay_width` dk or 1).
+// What is handed from delta_prep to the recurrence is the LOSS 1 - decay, from expm1: a decay next to one, rounded to a
+// float at every token, drifts over a thousand tokens of a state that forgets slowly.
 // The flat batch holds prompt portions beside single tokens: request r owns rows cu_q[r] .. cu_q[r+1]-1 and row
 // state_slots[r] of the state tensors, so a prompt may be cut anywhere.
 #include "common.cuh"
@@ -25,8 +27,8 @@ __device__ __forceinline__ float softplusf_(float x) { return fmaxf(x, 0.f) + lo
 constexpr int DELTA_MAX_TAPS = 16;
 
 // x [n, >= channels] at x_stride: the projections' output, q | k | v channels first (qk_cols = 2 * kv_heads * dk,
-// then heads * dv).  Outputs fp32: qk [n, qk_cols], v [n, heads * dv], g [n, heads * decay_width] (a_raw
-// and dt_bias alike), beta [n, heads].
+// then heads * dv).  Outputs fp32: qk [n, qk_cols], v [n, heads * dv], g [n, heads * decay_width] (the
+// losses 1 - decay; a_raw and dt_bias alike), beta [n, heads].
 // The work of a token is cut into units, one warp each: a q or k head (convolution, SiLU, unit norm: dk channels),
 // or a v head (dv channels) together with that head's decays and beta.  grid.y blocks share a token's units, so a
 // step of few tokens still fills the SMs.  `single` says that every request brings exactly one token: the thread
@@ -94,7 +96,7 @@ delta_prep_kernel(const T* __restrict__ x, int64_t x_stride, const float* __rest
       const float rate = -expf(A_log[h]);
       for (int c = lane; c < decay_width; c += 32) {
         const int hc = h * decay_width + c;
-        g[(int64_t)i * heads * decay_width + hc] = expf(rate * softplusf_(a_raw[(int64_t)i * a_stride + hc] + dt_bias[hc]));
+        g[(int64_t)i * heads * decay_width + hc] = -expm1f(rate * softplusf_(a_raw[(int64_t)i * a_stride + hc] + dt_bias[hc]));
       }
       if (lane == 0) beta[(int64_t)i * heads + h] = sigmoidf_(b_raw[(int64_t)i * b_stride + h]);
     }
@@ -270,7 +272,7 @@ delta_rule_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
       float pk[ACC] = {}, pq[ACC] = {};
 #pragma unroll
       for (int e = 0; e < DPT; ++e) {
-        S[e] *= gg[HEAD ? 0 : e];
+        S[e] = fmaf(-gg[HEAD ? 0 : e], S[e], S[e]);
         pk[e % ACC] = fmaf(S[e], kk[e], pk[e % ACC]);
         pq[e % ACC] = fmaf(S[e], qq[e], pq[e % ACC]);
       }

@@ -289,7 +289,8 @@ def delta_prep(x: torch.Tensor, conv_weight: torch.Tensor, conv_state: torch.Ten
     ``[n, heads]``: one per head) and ``beta_raw [n, heads]`` are fp32, rows may be slices: ``g = exp(-exp(A_log[h]) *
     softplus(decay_raw + dt_bias))``, ``beta = sigmoid(beta_raw)``.
     ``max_q_len`` 1 says that every request brings one token: the state is then brought up to date by the same
-    kernel.  Returns ``(qk [n, 2 * kv_heads * dk], v [n, heads * dv], g [n, heads * dk or heads], beta [n, heads])``."""
+    kernel.  Returns ``(qk [n, 2 * kv_heads * dk], v [n, heads * dv], g [n, heads * dk or heads], beta [n, heads])``;
+    the third is ``1 - g``, formed without the rounding a ``g`` next to one would carry."""
     _rows(x, "x")
     _rows(decay_raw, "decay_raw", torch.float32)
     _rows(beta_raw, "beta_raw", torch.float32)
@@ -320,7 +321,7 @@ def delta_prep(x: torch.Tensor, conv_weight: torch.Tensor, conv_state: torch.Ten
 def delta_rule(qk: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
                cu_q: torch.Tensor, state_slots: torch.Tensor, num_requests: int, heads: int, kv_heads: int, dk: int,
                dv: int, max_q_len: int = 0) -> torch.Tensor:
-    """Per (request, head), token after token: ``S <- diag(g) S`` (``g`` a number per key channel, or per head), ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
+    """Per (request, head), token after token: ``S <- diag(g) S`` (a number per key channel, or per head), ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
     ``o = S^T q`` (the read-out sees the token's own write).  Operands as ``delta_prep`` returns them; head ``h``
     uses the q and k of head ``h // (heads / kv_heads)``.  ``state [slots, heads, dv, dk]`` fp32 (one row per value
     column) is updated in place.  Returns fp32 ``[n, heads * dv]``."""
