@@ -9,7 +9,7 @@
 // model's output (depth_norm).  `value` may arrive as unsummed fp32 splits of a product (summed in ascending order
 // and rounded to T first).  Everything is fp32 but `value` and `out`.
 //
-// A block takes CH consecutive tokens of one request.  Rows before them that the convolution reaches into belong to
+// A block takes CHUNK consecutive tokens of one request.  Rows before them that the convolution reaches into belong to
 // another block, which writes them; this block computes them again (the inputs are not written in place, so there is
 // no order between blocks).  The first block of a request reads the request's state and is also the one that brings
 // it up to date: it computes the request's last taps-1 rows again when they are not its own.
@@ -19,6 +19,8 @@
 namespace {
 constexpr int MAX_TAPS = 16;
 constexpr int ROWS_MAX = 48;
+constexpr int THREADS_MAX = 512;
+constexpr int CHUNK = 8;                 // tokens per block
 
 template <int VEC> __device__ __forceinline__ void ld(const float* p, float (&v)[VEC]) {
   if constexpr (VEC == 4) {
@@ -106,7 +108,7 @@ __device__ __forceinline__ float stage_row(const Joined<T>& j, float* xs, int64_
 template <typename T, int VEC>
 __device__ __forceinline__ float row_squares(const Joined<T>& j, int64_t at, int width, int first, int stride) {
   float ss = 0.f;
-#pragma unroll 2
+#pragma unroll 8
   for (int c = first; c < width; c += stride) {
     float v[VEC];
     joined_value<T, VEC>(j, nullptr, at, c, v);
@@ -116,28 +118,38 @@ __device__ __forceinline__ float row_squares(const Joined<T>& j, int64_t at, int
   return ss;
 }
 
-// x (and X, when the average asks for it) of one row's VEC columns.
+// What one row's VEC columns bring: the residual, the sublayer's result, the weighted sum of the earlier streams.
+template <int VEC>
+struct RowIn {
+  float r[VEC], v[VEC], s[VEC];
+};
 template <typename T, int VEC>
-__device__ __forceinline__ void joined_x(const Joined<T>& j, const float* staged, float inv, int64_t at, int c, bool has_value,
-                                         const float (&pw)[VEC], float (&X)[VEC], float (&x)[VEC]) {
-  ld<VEC>(j.resid + at + c, X);
-  if (has_value) {
-    float v[VEC];
-    joined_value<T, VEC>(j, staged, at, c, v);
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) X[e] = fmaf(v[e] * inv, pw[e], X[e]);
-  }
+__device__ __forceinline__ void fetch_row(const Joined<T>& j, const float* staged, int64_t at, int c, bool has_value,
+                                          RowIn<VEC>& in) {
+  ld<VEC>(j.resid + at + c, in.r);
+  if (has_value) joined_value<T, VEC>(j, staged, at, c, in.v);
   if (j.depth_w) {
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) x[e] = 0.f;
+    for (int e = 0; e < VEC; ++e) in.s[e] = 0.f;
 #pragma unroll 4
     for (int k = 0; k < j.count; ++k) {
       float s[VEC];
       ld<VEC>(j.streams + (int64_t)k * j.stream_stride + at + c, s);
       const float w = j.depth_w[k];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) x[e] = fmaf(w, s[e], x[e]);
+      for (int e = 0; e < VEC; ++e) in.s[e] = fmaf(w, s[e], in.s[e]);
     }
+  }
+}
+// X and x from it.
+template <typename T, int VEC>
+__device__ __forceinline__ void joined_x(const Joined<T>& j, const RowIn<VEC>& in, float inv, bool has_value,
+                                         const float (&pw)[VEC], float (&X)[VEC], float (&x)[VEC]) {
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) X[e] = has_value ? fmaf(in.v[e] * inv, pw[e], in.r[e]) : in.r[e];
+  if (j.depth_w) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[e] = in.s[e];
     const float w = j.depth_w[j.count];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) x[e] = fmaf(w, X[e], x[e]);
@@ -150,7 +162,7 @@ __device__ __forceinline__ void joined_x(const Joined<T>& j, const float* staged
 // conv_w: [taps, width], the last row multiplies the current token; conv_state: [slots, taps-1, width], oldest first.
 // TMAX >= taps: the window a thread keeps (what lies beyond `taps` is multiplied by zero).
 template <typename T, int TMAX, int VEC>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(THREADS_MAX)
 depth_conv_kernel(Joined<T> j, float* __restrict__ x_out, const float* __restrict__ conv_w, float* __restrict__ conv_state,
                   const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* __restrict__ out, int width,
                   int taps, int chunk) {
@@ -209,13 +221,18 @@ depth_conv_kernel(Joined<T> j, float* __restrict__ x_out, const float* __restric
         if (opens && tap < keep) ld<VEC>(cs + (int64_t)tap * width + c, win[k + 1 < TMAX ? k + 1 : k]);
       }
     }
-#pragma unroll 2
-    for (int i = 0; i < count; ++i) {
+    // a row's loads are issued a row ahead, before the stores of the row in hand
+    auto fetch = [&](int i, RowIn<VEC>& in) {
+      fetch_row<T, VEC>(j, j.parts ? xs + (int64_t)i * width : nullptr, (int64_t)(t0 + row_of(i)) * width, c, has_value, in);
+    };
+    RowIn<VEC> now, next;
+    fetch(0, now);
+    for (int i = 0; i < count; ++i, now = next) {
+      if (i + 1 < count) fetch(i + 1, next);
       const int row = row_of(i);
       const int64_t at = (int64_t)(t0 + row) * width;
       float X[VEC], x[VEC];
-      joined_x<T, VEC>(j, j.parts ? xs + (int64_t)i * width : nullptr, has_value ? inv_s[i] : 0.f, at, c, has_value, pw,
-                       X, x);
+      joined_x<T, VEC>(j, now, has_value ? inv_s[i] : 0.f, has_value, pw, X, x);
 #pragma unroll
       for (int k = 0; k + 1 < TMAX; ++k)
 #pragma unroll
@@ -267,8 +284,10 @@ depth_norm_kernel(Joined<T> j, const int* __restrict__ rows, const float* __rest
   float ss = 0.f;
   for (int c = first; c < width; c += stride) {
     float pw[VEC] = {}, X[VEC], x[VEC];
+    RowIn<VEC> in;
     if (has_value) ld<VEC>(j.post_w + c, pw);
-    joined_x<T, VEC>(j, j.parts ? xs : nullptr, inv, at, c, has_value, pw, X, x);
+    fetch_row<T, VEC>(j, j.parts ? xs : nullptr, at, c, has_value, in);
+    joined_x<T, VEC>(j, in, inv, has_value, pw, X, x);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ss = fmaf(x[e], x[e], ss);
     st<VEC>(xs + c, x);                                      // read back by the thread that wrote it
@@ -301,7 +320,7 @@ bool valid(const Joined<T>& j, int width) {
 }
 
 inline int threads_for(int width, int vec) {
-  return std::max(32, std::min(512, (width / vec + 31) / 32 * 32));
+  return std::max(32, std::min(THREADS_MAX, (width / vec + 31) / 32 * 32));
 }
 
 template <typename K>
@@ -318,7 +337,7 @@ int depth_conv_launch(Joined<T> j, float* x_out, const float* conv_w, float* con
   if (!valid(j, width) || taps < 1 || taps > MAX_TAPS || num_requests > 65535 || conv_w == nullptr || out == nullptr ||
       (taps > 1 && conv_state == nullptr) || x_out == j.resid)
     return (int)cudaErrorInvalidValue;
-  const int chunk = max_q_len == 1 ? std::max(1, taps - 1) : std::max(8, taps - 1);
+  const int chunk = max_q_len == 1 ? std::max(1, taps - 1) : std::max(CHUNK, taps - 1);
   const int rows_most = max_q_len == 1 ? 1 : chunk + taps - 1;
   const size_t smem = j.parts ? sizeof(float) * (size_t)rows_most * width : 0;
   if (rows_most > ROWS_MAX || smem > 200 * 1024) return (int)cudaErrorInvalidValue;

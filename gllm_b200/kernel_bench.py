@@ -592,7 +592,9 @@ def distance_attention(tokens=2048, batch=1, context=0, hq=32, hkv=8, dk=64, dv=
     flops = 2.0 * (dk + dv) * hq * batch * _visible(tokens, context, window, keep)
     keys = min(context + tokens, window + keep + tokens) if window else context + tokens
     nbytes = batch * keys * hkv * (dk + dv) * 2 + n * hq * (dk + dv) * 2
-    return _result("distance_attention (mma.sync)" if mma else "distance_attention (CUDA cores)", us, peaks, shape, nbytes,
+    tcgen05 = mma and tokens >= distance.TMEM_MIN_Q_LEN and distance.takes_tmem(hq, hkv, dk, dv, block_size, 1001)
+    kind = "tcgen05" if tcgen05 else ("mma.sync" if mma else "CUDA cores")
+    return _result(f"distance_attention ({kind})", us, peaks, shape, nbytes,
                    flops)
 
 
