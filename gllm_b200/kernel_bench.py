@@ -598,6 +598,23 @@ def distance_attention(tokens=2048, batch=1, context=0, hq=32, hkv=8, dk=64, dv=
                    flops)
 
 
+def rope_store(tokens=2048, batch=1, context=0, hq=32, hkv=8, d=64, block_size=16, iters=5, peaks=None):
+    """Rotation of q and k and the store of k and v: the kernel before Llama's attention."""
+    from gllm_b200 import ops
+
+    b = _Batch(batch, tokens, context)
+    pool, table = _paged_cache(batch, context + tokens, hkv, d, block_size)
+    n = batch * tokens
+    qkv = torch.randn(n, (hq + 2 * hkv) * d, device="cuda").to(torch.bfloat16)
+    page = table[b.token_row.long(), (b.positions // block_size).long()]
+    slots = (page * block_size + b.positions % block_size).to(torch.int32)
+    freq = torch.rand(d // 2, device="cuda")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    us = _time(lambda: ops.rope_store(qkv, b.positions, freq, slots, pool, hq, hkv, d, d), iters, flush)
+    return _result("rope_store", us, peaks, dict(tokens=tokens, batch=batch, heads=hq, kv_heads=hkv, head_dim=d),
+                   n * 2 * (hq + 2 * hkv) * d * 2)
+
+
 def depth_conv(tokens=2048, batch=1, hidden=2048, taps=4, streams=0, splits=0, iters=5, peaks=None):
     """The kernel between two sublayers: norm and add of the sublayer's result (a tensor, or ``splits`` unsummed fp32
     parts), the average over ``streams`` earlier streams (0: none), the convolution over time."""
@@ -626,6 +643,7 @@ def depth_conv(tokens=2048, batch=1, hidden=2048, taps=4, streams=0, splits=0, i
 KERNELS = {
     "distance_attention": distance_attention,
     "depth_conv": depth_conv,
+    "rope_store": rope_store,
     "differential_attention": differential_attention,
     "step_sized_recurrence": step_sized_recurrence,
     "add_dyt": add_dyt,

@@ -194,7 +194,7 @@ PLANS = [[(0, 37), (1, 9)], [(0, 2), (1, 1)], [(0, 1), (1, 1)], [(0, 64), (1, 30
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,size,keep,far,rows,page", [
     (4, 2, 16, 24, 40, 5, 60, 12, 4), (3, 1, 8, 40, 17, 33, 25, 7, 8), (6, 2, 64, 64, 64, 0, 300, 16, 16),
     (8, 1, 128, 128, 100, 20, 90, 32, 16), (2, 2, 32, 8, None, 0, 40.5, 6, 32), (5, 5, 72, 120, 1, 70, 12, 8, 16),
-    (16, 1, 48, 32, 63, 64, 500, 10, 16), (12, 1, 24, 16, 65, 1, 33, 5, 8)])
+    (16, 1, 56, 40, 63, 64, 500, 10, 16), (12, 1, 24, 16, 65, 1, 33, 5, 8)])
 def test_attention_with_a_bias_by_distance(cores, heads, kv_heads, dim, vdim, size, keep, far, rows, page):
     """Biases, norms, the mix of values, the store into shuffled pages and the attention of two requests fed in portions
     and single tokens, against the plain functions.  One early key stands out for every query (inside the kept tokens
@@ -320,7 +320,7 @@ def test_values_of_the_first_layer_are_kept():
 
 
 @pytest.mark.parametrize("cores", ["cuda", "tensor"])
-@pytest.mark.parametrize("heads,dim,rot,rank,size,page", [(4, 16, 8, 40, 33, 4), (3, 8, 16, 96, 64, 16), (16, 32, 32, 128, 31, 8),
+@pytest.mark.parametrize("heads,dim,rot,rank,size,page", [(4, 16, 8, 40, 33, 4), (3, 8, 16, 88, 64, 16), (16, 32, 32, 128, 31, 8),
                                                          (8, 64, 64, 512, 100, 16), (1, 24, 24, 72, 1, 16), (20, 8, 8, 200, 65, 8),
                                                          (2, 16, 16, 64, None, 16)])
 def test_latent_attention_in_a_window(cores, heads, dim, rot, rank, size, page):
