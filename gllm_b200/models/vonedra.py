@@ -88,6 +88,8 @@ def build_vonedra_spec(cfg: VonedraConfig) -> ModelSpec:
             parts["feed_forward"] = PartSpec("swiglu", dict(hidden_size=width, intermediate_size=layer.mlp["ff"]),
                                              {n: f"{p}.mlp.{n}" for n in ("gate", "up", "down")})
             parts["feed_forward_norm"] = norm(f"{p}.norm2")
+        else:                                   # a checkpoint may hold them all the same
+            ignorable += [f"{p}.norm2", f"{p}.canon2"]
         # the embedding output, the layers before this one, and this one
         parts["depth_average"] = PartSpec("depth_average", dict(streams=i + 2), {"weight": f"{p}.dwa"})
         layers.append(LayerSpec("result_norm", parts))

@@ -74,7 +74,7 @@ def test_spec_parts_and_what_they_ask_of_the_cache():
     from gllm_b200.models.decoder import DecoderModel
 
     spec = architecture_for("Vonedra").build_spec(load_config(copy.deepcopy(VONEDRA["A"])))
-    assert spec.depth_streams and spec.head_name == "head" and spec.ignorable_names == ("l2.mix.vmix",)
+    assert spec.depth_streams and spec.head_name == "head" and spec.ignorable_names == ("l2.mix.vmix", "l2.norm2", "l2.canon2")
     assert [l.mixer.params.get("value_mix") for l in spec.layers] == ["first", None, None, None, "mixed"]
     assert [l.depth_average.params["streams"] for l in spec.layers] == [2, 3, 4, 5, 6]
     assert "feed_forward" not in spec.layers[2].parts
