@@ -1,10 +1,10 @@
 """The cache manager.
 
 Layers whose mixers ask for the same kind of pages (kv heads, head size,
-window) form a *group*: one page id addresses that page in every layer of the
-group, and each request has one block list per group.  Groups with a window
-give pages back as soon as the window has moved past them (but for the pages of the first tokens, where a mixer
-keeps seeing those); all groups give
+window, chunks) form a *group*: one page id addresses that page in every layer of the
+group, and each request has one block list per group.  Groups with a window (or with chunks)
+give pages back as soon as the window has moved past them (the chunk has ended; but for the pages of the first tokens,
+where a mixer keeps seeing those); all groups give
 everything back when a request ends.  Freed pages are handed out again.
 Beside the pages, every live request holds one *state slot*, the row of its
 block tables and of every fixed-size state tensor a mixer declared.
@@ -71,7 +71,8 @@ class CacheManager:
         allocate_pools: bool = True,
     ):
         """``requirements``: per plan entry ``(KVPageRequirement | None,
-        StateRequirement | None, reads_cache_of | None)``."""
+        StateRequirement | None, reads_cache_of | None)``.  An entry that reads another's pages shares that entry's
+        states when it names none, and keeps its own when it does."""
         self.block_size = int(block_size)
         self.num_blocks = int(num_blocks)
         self.max_batch_size = int(max_batch_size)
@@ -85,6 +86,7 @@ class CacheManager:
         self._entry_group: list[int | None] = []
         self._entry_layer: list[int | None] = []
         self._entry_writes: list[bool] = []
+        self._entry_owns_states: list[bool] = []
         self._states: list[tuple[torch.Tensor, ...] | None] = []
         self._state_reqs: list[tuple[StateRequirement, ...] | None] = []
         by_req: dict[KVPageRequirement, CacheGroup] = {}
@@ -95,8 +97,12 @@ class CacheManager:
                 self._entry_group.append(self._entry_group[reads])
                 self._entry_layer.append(self._entry_layer[reads])
                 self._entry_writes.append(False)
-                self._states.append(self._states[reads])
-                self._state_reqs.append(None)
+                self._entry_owns_states.append(state is not None)
+                if state is None:
+                    self._states.append(self._states[reads])
+                    self._state_reqs.append(None)
+                else:
+                    self._add_states(state, allocate_pools)
                 continue
             if kv is not None:
                 group = by_req.get(kv)
@@ -111,17 +117,8 @@ class CacheManager:
                 self._entry_group.append(None)
                 self._entry_layer.append(None)
             self._entry_writes.append(True)
-            # a mixer may ask for one state tensor or for several
-            wanted = () if state is None else (tuple(state) if isinstance(state, (tuple, list)) else (state,))
-            self._state_reqs.append(wanted or None)
-            if wanted and allocate_pools:
-                # one row more than there are slots: the null row, for rows that pad a batch
-                self._states.append(tuple(
-                    torch.zeros((self.max_batch_size + 1, *s.shape), dtype=s.dtype, device=self.device)
-                    for s in wanted
-                ))
-            else:
-                self._states.append(None)
+            self._entry_owns_states.append(True)
+            self._add_states(state, allocate_pools)
         for g in self.groups:
             r = g.requirement
             # One page more than the allocator hands out: the *null page* (id num_blocks).
@@ -139,6 +136,17 @@ class CacheManager:
             g.block_table[self.max_batch_size].fill_(self.num_blocks)
             g.block_table_host = np.full((self.max_batch_size + 1, self.max_blocks_per_request), -1, dtype=np.int32)
             g.block_table_host[self.max_batch_size] = self.num_blocks
+
+    def _add_states(self, state, allocate: bool) -> None:
+        # a mixer may ask for one state tensor or for several
+        wanted = () if state is None else (tuple(state) if isinstance(state, (tuple, list)) else (state,))
+        self._state_reqs.append(wanted or None)
+        if wanted and allocate:
+            # one row more than there are slots: the null row, for rows that pad a batch
+            self._states.append(tuple(
+                torch.zeros((self.max_batch_size + 1, *s.shape), dtype=s.dtype, device=self.device) for s in wanted))
+        else:
+            self._states.append(None)
 
     @property
     def null_page(self) -> int:
@@ -167,7 +175,7 @@ class CacheManager:
         rc = RequestCache(request_id, slot, 0, {g.index: [] for g in self.groups})
         self.requests[request_id] = rc
         for idx, states in enumerate(self._states):
-            if states is not None and self._entry_writes[idx]:
+            if states is not None and self._entry_owns_states[idx]:
                 for state in states:
                     state[slot].zero_()
         return rc
@@ -183,7 +191,7 @@ class CacheManager:
 
     def pages_for_admission(self, n_tokens: int) -> dict[int, int]:
         """Pages each group needs for the first ``n_tokens`` tokens of a request that holds nothing yet
-        (a window group gives pages back only after the step that stored them)."""
+        (a group with a window or chunks gives pages back only after the step that stored them)."""
         return {g.index: -(-n_tokens // g.block_size) for g in self.groups}
 
     def can_append(self, request_id, n_new: int) -> bool:
@@ -233,13 +241,12 @@ class CacheManager:
         rc = self.requests[request_id]
         rc.num_tokens += n_new
         for group in self.groups:
-            w = group.window
-            if w is None:
+            if not group.requirement.bounded:
                 continue
             blocks = rc.blocks[group.index]
             kept = -(-group.requirement.keep_first // self.block_size)      # pages of the first tokens stay
-            # the next token sits at position >= num_tokens and sees keys >= num_tokens - w + 1
-            dead = max(0, (rc.num_tokens - w + 1)) // self.block_size
+            # the next token sits at position >= num_tokens
+            dead = group.requirement.first_needed(rc.num_tokens) // self.block_size
             release = []
             for b in range(kept, min(dead, len(blocks))):
                 if blocks[b] >= 0:

@@ -38,6 +38,7 @@ def _ensure_builtin_loaded() -> None:
     import gllm_b200.models.guvetar  # noqa: F401
     import gllm_b200.models.llama  # noqa: F401
     import gllm_b200.models.mifidra  # noqa: F401
+    import gllm_b200.models.pifelix  # noqa: F401
     import gllm_b200.models.rulunex  # noqa: F401
     import gllm_b200.models.sazisun  # noqa: F401
     import gllm_b200.models.vonedra  # noqa: F401

@@ -51,7 +51,6 @@ decode_split_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride,
   // chunk-major: all (request, kv head) pairs of chunk 0 come first, and the chunks past every request's end (the
   // grid is sized for the longest sequence of the step's bucket) come last: 0.913 -> 0.900 ms per decode step at
   // batch 8, 0.780 -> 0.765 at batch 1, against the chunks of one request side by side
-  const int split = blockIdx.y;
   const int group = hq / hkv;
   const int head_tiles = (group + ROWS - 1) / ROWS;
   const int n = (int)blockIdx.x / (hkv * head_tiles), by = (int)blockIdx.x - n * (hkv * head_tiles);
@@ -60,10 +59,12 @@ decode_split_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride,
   const int heads = min(ROWS, group - tile_idx * ROWS);
 
   const int qpos = positions[n];
-  const int kstart = window > 0 ? max(0, qpos - window + 1) : 0;
+  const int kstart = first_visible_key(qpos, window);
+  // blockIdx.y counts from the chunk of the query's first visible key
+  const int part = blockIdx.y, split = kstart / S::CHUNK + part;
   const int c0 = max(split * S::CHUNK, kstart);
   const int c1 = min((split + 1) * S::CHUNK, qpos + 1);
-  float* my_ml = part_ml + (((int64_t)n * hq + h0) * num_chunks + split) * 2;
+  float* my_ml = part_ml + (((int64_t)n * hq + h0) * num_chunks + part) * 2;
   if (c0 >= c1) {                                       // nothing of this chunk is visible
     pdl_wait();
     if (threadIdx.x < heads) {
@@ -247,7 +248,7 @@ decode_split_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride,
       acc += all_o[((size_t)w * ROWS + row) * D + d] * f;
       ll += red_l[w][row] * f;
     }
-    part_o[(((int64_t)n * hq + h0 + row) * num_chunks + split) * D + d] = acc;
+    part_o[(((int64_t)n * hq + h0 + row) * num_chunks + part) * D + d] = acc;
     if (d == 0) {
       float* ml = my_ml + (int64_t)row * num_chunks * 2;
       ml[0] = mm;                                       // in units of log2
@@ -257,8 +258,8 @@ decode_split_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride,
 }
 
 // Merges the partial results of one (request, query head) in ascending order, in one pass (running
-// maximum, sum and output).  Only the chunks that can hold a visible key are read: those of the keys
-// kstart .. qpos, `per_span` consecutive chunks for every `span_keys` keys.
+// maximum, sum and output).  Only the chunks that can hold a visible key are read, counted from the one of the first
+// visible key: those of the keys kstart .. qpos, `per_span` consecutive chunks for every `span_keys` keys.
 template <int D>
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                      __nv_bfloat16* __restrict__ out, int64_t out_stride, int hq, int num_chunks,
@@ -266,9 +267,8 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   pdl_trigger();
   const int n = blockIdx.y, h = blockIdx.x, d = threadIdx.x;
   const int qpos = positions[n];                          // a step input: older than the step's kernels
-  const int kstart = window > 0 ? max(0, qpos - window + 1) : 0;
-  const int first = (kstart / span_keys) * per_span;
-  const int last = min(num_chunks, (qpos / span_keys + 1) * per_span);
+  const int kstart = first_visible_key(qpos, window);
+  const int first = 0, last = min(num_chunks, (qpos / span_keys - kstart / span_keys + 1) * per_span);
   pdl_wait();
   const float* ml = part_ml + ((int64_t)n * hq + h) * num_chunks * 2;
   const float* po = part_o + ((int64_t)n * hq + h) * num_chunks * D;
@@ -333,7 +333,8 @@ GLLM_API int gllm_attention_decode_chunk(int d) {
 // Query token i of the call is row i of q / out / positions / token_row.
 // Scratch the caller provides: part_o  [num_queries * hq * num_chunks * d] floats,
 //                              part_ml [num_queries * hq * num_chunks * 2] floats,
-// num_chunks = ceil(longest sequence / gllm_attention_decode_chunk(d)) (or more).
+// num_chunks = the chunks of gllm_attention_decode_chunk(d) keys that hold a query's visible keys, at most (or more):
+// ceil(longest sequence / chunk), fewer with a window.  window: see first_visible_key.
 GLLM_API int gllm_attention_decode_bf16(const __nv_bfloat16* q, int64_t q_stride, __nv_bfloat16* out,
                                         int64_t out_stride, const __nv_bfloat16* cache, const int* block_table,
                                         int bt_stride, const int* positions, const int* token_row,

@@ -71,7 +71,7 @@ __host__ __device__ inline StreamPlan make_plan(int d, int hq, int hkv, int bloc
 }
 
 struct WorkItem {
-  int n, span, qpos, c0, c1;
+  int n, part, span, qpos, c0, c1;     // part: the span counted from the one of the first visible key
   bool empty;
 };
 
@@ -126,10 +126,11 @@ decode_stream_kernel(const __grid_constant__ CUtensorMap map_kv, const __nv_bflo
   // ones that hold the newest keys last.
   auto item_of = [&](int w) -> WorkItem {
     WorkItem it;
-    it.span = w / num_queries;
-    it.n = w - it.span * num_queries;
+    it.part = w / num_queries;
+    it.n = w - it.part * num_queries;
     it.qpos = it.n < MAXQ ? s_qpos[it.n] : positions[it.n];
-    const int kstart = window > 0 ? max(0, it.qpos - window + 1) : 0;
+    const int kstart = first_visible_key(it.qpos, window);
+    it.span = kstart / SPAN + it.part;
     it.c0 = max(it.span * SPAN, kstart);
     it.c1 = min((it.span + 1) * SPAN, it.qpos + 1);
     it.empty = it.c0 >= it.c1;
@@ -238,7 +239,7 @@ decode_stream_kernel(const __grid_constant__ CUtensorMap map_kv, const __nv_bflo
       const WorkItem item = item_of(w);
       if (item.empty) {                                   // nothing of this span is visible
         if (working && lane < heads) {
-          float* ml = part_ml + (((int64_t)item.n * hq + h0 + lane) * chunks_total + item.span * plan.pps + slot) * 2;
+          float* ml = part_ml + (((int64_t)item.n * hq + h0 + lane) * chunks_total + item.part * plan.pps + slot) * 2;
           ml[0] = -INFINITY;
           ml[1] = 0.f;
         }
@@ -375,7 +376,7 @@ decode_stream_kernel(const __grid_constant__ CUtensorMap map_kv, const __nv_bflo
       if (!ok) break;
       // ---- this warp's partial result of the span: one chunk per (span, page slot)
       if (working) {
-        const int chunk = item.span * plan.pps + slot;
+        const int chunk = item.part * plan.pps + slot;
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int row = g8 + 8 * i;
@@ -397,8 +398,8 @@ decode_stream_kernel(const __grid_constant__ CUtensorMap map_kv, const __nv_bflo
 }
 
 // Merges the partial results of one (request, query head) in ascending order, in one pass (running
-// maximum, sum and output).  Only the chunks that can hold a visible key are read: those of the keys
-// kstart .. qpos, `per_span` consecutive chunks for every `span_keys` keys.
+// maximum, sum and output).  Only the chunks that can hold a visible key are read, counted from the one of the first
+// visible key: those of the keys kstart .. qpos, `per_span` consecutive chunks for every `span_keys` keys.
 template <int D>
 __global__ void decode_stream_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                      __nv_bfloat16* __restrict__ out, int64_t out_stride, int hq, int num_chunks,
@@ -406,9 +407,8 @@ __global__ void decode_stream_merge_kernel(const float* __restrict__ part_o, con
   pdl_trigger();
   const int n = blockIdx.y, h = blockIdx.x, d = threadIdx.x;
   const int qpos = positions[n];                          // a step input: older than the step's kernels
-  const int kstart = window > 0 ? max(0, qpos - window + 1) : 0;
-  const int first = (kstart / span_keys) * per_span;
-  const int last = min(num_chunks, (qpos / span_keys + 1) * per_span);
+  const int kstart = first_visible_key(qpos, window);
+  const int first = 0, last = min(num_chunks, (qpos / span_keys - kstart / span_keys + 1) * per_span);
   pdl_wait();
   const float* ml = part_ml + ((int64_t)n * hq + h) * num_chunks * 2;
   const float* po = part_o + ((int64_t)n * hq + h) * num_chunks * D;
@@ -518,7 +518,7 @@ GLLM_API int gllm_attention_decode_stream_parts(int d, int hq, int hkv, int bloc
 }
 
 // Query token i of the call is row i of q / out / positions / token_row.  num_spans =
-// ceil(longest sequence / 128) (or more); with parts = gllm_attention_decode_stream_parts(...) the
+// ceil(longest sequence / 128), fewer with a window (the spans that hold a query's visible keys; or more); with parts = gllm_attention_decode_stream_parts(...) the
 // caller provides scratch: part_o  [num_queries * hq * num_spans * parts * d] floats,
 //                          part_ml [num_queries * hq * num_spans * parts * 2] floats.
 // q and the cache layer must be 16-byte aligned, q_stride a multiple of 8.

@@ -53,7 +53,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, __nv_bfloa
   const int g8 = lane >> 2, t4 = lane & 3;
 
   const int pos_first = ctx + t0, pos_last = ctx + t0 + t_count - 1;
-  const int kv_lo = window > 0 ? max(0, pos_first - window + 1) : 0;
+  const int kv_lo = first_visible_key(pos_first, window);
   const int tile_first = kv_lo / BN, tile_last = pos_last / BN;
 
   const int64_t head_elems = (int64_t)block_size * D;
@@ -95,7 +95,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, __nv_bfloa
   cp_async_commit();
 
   // per-thread rows: rr0 = warp*16 + g8 and rr0 + 8
-  int qpos[2];
+  int qpos[2], lo[2];
   bool row_ok[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
@@ -103,6 +103,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, __nv_bfloa
     const int tl = rr / gp;
     row_ok[i] = tl < t_count;
     qpos[i] = pos_first + tl;
+    lo[i] = first_visible_key(qpos[i], window);
   }
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[D / 8][4];
@@ -156,7 +157,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, __nv_bfloa
     }
     // ---- mask, online softmax (rows g8 and g8 + 8 of the warp's 16).  The maximum is kept in raw
     // score units; the scale enters through the exponent's FMA: p = 2^(s*c - m*c), c = scale*log2(e)
-    const bool need_mask = (kv0 + BN - 1 > pos_first) || (window > 0) || (t_count < qt);
+    const bool need_mask = (kv0 + BN - 1 > pos_first) || (window != 0) || (t_count < qt);
     float mx[2] = {-INFINITY, -INFINITY};
     if (need_mask) {
 #pragma unroll
@@ -165,7 +166,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, __nv_bfloa
         for (int e = 0; e < 4; ++e) {
           const int i = e >> 1;
           const int key = kv0 + nt * 8 + 2 * t4 + (e & 1);
-          const bool hidden = !row_ok[i] || key > qpos[i] || (window > 0 && key <= qpos[i] - window);
+          const bool hidden = !row_ok[i] || key > qpos[i] || key < lo[i];
           if (hidden) s[nt][e] = -INFINITY;
         }
     }

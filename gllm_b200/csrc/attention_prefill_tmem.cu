@@ -217,7 +217,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   const int t_count = has_rows ? min(qt, q_len - t0) : 0;
   const int ctx = ctx_lens[r];
   const int pos_first = ctx + t0, pos_last = ctx + t0 + t_count - 1;
-  const int kv_lo = window > 0 ? max(0, pos_first - window + 1) : 0;
+  const int kv_lo = first_visible_key(pos_first, window), lo_last = first_visible_key(pos_last, window);
   const int tile_last = pos_last / BN;
   const int keep = BIAS && window > 0 ? dist.keep_first : 0;          // keys below this one are seen beside the window
   int tile_first = kv_lo / BN, n_kept = (keep + BN - 1) / BN;         // tiles of those keys come first
@@ -386,6 +386,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // (with a bias the scores are brought to log2 units when they are read)
     const float sl = BIAS ? 1.f : scale_log2;
     const float* my_bias = BIAS ? table + g * dist.table_ld + BIAS_PAD : nullptr;
+    const int lo = first_visible_key(qpos, window);     // this row's first visible key
     bool ok = true;
     // Head size 64: one pass per tile.  The probabilities are taken against the reference maximum the row
     // already has while the tile's maximum is found on the side; only when some row's maximum has outgrown
@@ -401,7 +402,6 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       // keys this row sees in the tile: lo <= key <= hi (hi < lo: none)
       const int hi = row_ok ? qpos : -1;
-      const int lo = window > 0 ? max(0, qpos - window + 1) : 0;
       const unsigned span = hi >= lo ? (unsigned)(hi - lo) : 0u;
       const int lo_eff = hi >= lo ? lo : 0x7fffff00;     // no key passes when the row sees nothing
       // Each chunk of 32 keys is, for all rows of the CTA alike: seen by no row (nothing is computed, its
@@ -412,7 +412,7 @@ prefill_tmem_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       for (int ci = 0; ci < HK / 32; ++ci) {
         const int k0 = kv0 + ci * 32;
         const bool none = k0 > pos_last || (k0 + 31 < kv_lo && (!BIAS || k0 >= keep));
-        const bool all = k0 + 31 <= pos_first && (window <= 0 || k0 >= pos_last - window + 1 || (BIAS && k0 + 31 < keep));
+        const bool all = k0 + 31 <= pos_first && (k0 >= lo_last || (BIAS && k0 + 31 < keep));
         cls[ci] = none ? CHUNK_SKIP : all ? CHUNK_FAST : CHUNK_MASK;
       }
       // the tile's scores -> (maximum) and/or (probabilities in tensor memory, their sums)

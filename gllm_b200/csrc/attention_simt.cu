@@ -8,9 +8,9 @@
 // (gllm/model/layers/attention.py:165-173,
 // gllm/ops/attention/reference_attention.py:40-48): no bias tensor, no score
 // tensor and no gathered copy exist here.  A token at position p of a request
-// sees the keys at positions max(0, p - window + 1) .. p of that request
-// (window <= 0: all of them), found through the request's row of the block
-// table.  Scores, the running maximum, the running sum and the output
+// sees the keys at positions first_visible_key(p, window) .. p of that request
+// (window 0: all of them; < 0: those of its own chunk), found through the
+// request's row of the block table.  Scores, the running maximum, the running sum and the output
 // accumulator are fp32; the order of accumulation depends only on absolute
 // key positions (blocks of 32 keys aligned to multiples of 32), never on how
 // the request was cut into steps or on the rest of the batch.
@@ -43,7 +43,7 @@ attention_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__
   for (int i = lane; i < d; i += 32) q_s[warp][i] = to_float(qv[i]);
   __syncwarp();
 
-  const int kstart = window > 0 ? max(0, qpos - window + 1) : 0;
+  const int kstart = first_visible_key(qpos, window);
   const size_t head_elems = (size_t)block_size * d;
   const size_t page_elems = (size_t)2 * hkv * head_elems;
   float m = -INFINITY, l = 0.f;

@@ -41,6 +41,14 @@ __device__ __forceinline__ float gate_act(float g, float u, const GateAct& a) {
   return g / (1.0f + __expf(-a.slope * g)) * (u + a.offset);
 }
 
+// The first key position a query at position p sees, whatever kind of bound the layer has: `window` > 0 keeps the last
+// `window` positions, `window` < 0 cuts the sequence into chunks of -window positions counted from position 0 and keeps
+// those of the query's own chunk, 0 keeps all.  It never falls as p grows.
+__device__ __forceinline__ int first_visible_key(int p, int window) {
+  if (window > 0) return max(0, p - window + 1);
+  return window < 0 ? p / -window * -window : 0;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

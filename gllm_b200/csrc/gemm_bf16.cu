@@ -74,6 +74,7 @@ struct Groups {
   const int* group_of_tile;
   const int* num_tiles;
   int group_rows;
+  const float* row_scale;      // GATED: a number per row of X that multiplies the row's products ahead of the activation, or null
 };
 // Work item w of a launch.  Normal: neighbouring CTAs share a weight tile.  Swapped:
 // neighbouring CTAs take the K ranges of the same weight rows.
@@ -279,6 +280,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
         if (!SWAPPED) {
           // this thread's token row holds, per 128 columns, 64 gates then their 64 ups
           const int m = item.a_row0 + row;
+          const float rs = groups.row_scale != nullptr && m < M ? groups.row_scale[m] : 1.f;
 #pragma unroll 1
           for (int c2 = 0; c2 < BN / 2; c2 += 16) {
             const int gate_col = (c2 / 64) * 128 + (c2 % 64);
@@ -289,7 +291,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             if (m < M && f0 < n_out) {
               float y[16];
 #pragma unroll
-              for (int i = 0; i < 16; ++i) y[i] = gate_act(g[i], u[i], act);
+              for (int i = 0; i < 16; ++i) y[i] = gate_act(g[i] * rs, u[i] * rs, act);
               OutT* dst = out + (int64_t)m * ldo + f0;
               if (f0 + 16 <= n_out && sizeof(OutT) == 2 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
                 uint4 p0, p1;
@@ -492,7 +494,7 @@ template <int BN, bool SWAPPED, typename OutT, bool GATED>
 int umma_launch(const __nv_bfloat16* X, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int64_t ldx,
                 int64_t ldw, int64_t ldo, int splits, float* partial, int* tickets, int reduce_in_kernel, int* status,
                 cudaStream_t stream, int accumulate = 0, GateAct act = GateAct{1.f, 0.f, 0.f},
-                Groups groups = Groups{nullptr, nullptr, 0}, int w_rows = 0) {
+                Groups groups = Groups{nullptr, nullptr, 0, nullptr}, int w_rows = 0) {
   using S = Shape<BN>;
   CUtensorMap map_a, map_b;
   if (w_rows <= 0) w_rows = N;                 // grouped: the weight's map covers the rows of all groups
@@ -636,18 +638,21 @@ GLLM_API int gllm_gemm_bf16_accumulate(const __nv_bfloat16* X, const __nv_bfloat
 
 // Grouped product: the rows of X [rows, K] come in tiles of 128 that each belong to one group (``group_of_tile``,
 // ``num_tiles`` on the device); group g multiplies by W[g] of W [groups, N, K].  gated != 0: W[g]'s rows are blocks of
-// 64 gate rows and the 64 up rows of the same features and out is bf16 [rows, N / 2] = silu(gate) * up; otherwise out
-// is fp32 [rows, N].  Rows of tiles behind ``num_tiles[0]`` are neither read nor written; a row of X that no pair
+// 64 gate rows and the 64 up rows of the same features and out is bf16 [rows, N / 2], the gated activation of the two
+// (slope, limit, offset as gllm_gemm_bf16_gated takes them; row_scale, null or [rows]: gate and up are multiplied by the
+// row's number first); otherwise out is fp32 [rows, N].  Rows of tiles behind ``num_tiles[0]`` are neither read nor written; a row of X that no pair
 // owns gives a row of out that nobody reads (rows do not mix).
 GLLM_API int gllm_gemm_bf16_grouped(const __nv_bfloat16* X, const __nv_bfloat16* W, void* out, int gated, int rows, int N,
                                     int K, int groups, const int* group_of_tile, const int* num_tiles, int wide,
-                                    int* status, cudaStream_t stream) {
+                                    const float* row_scale, float slope, float limit, float offset, int* status,
+                                    cudaStream_t stream) {
   if (rows <= 0 || N <= 0 || groups <= 0) return 0;
   if (rows % BM || K <= 0 || K % 8 || (gated && N % 128) || (reinterpret_cast<uintptr_t>(X) & 15) ||
       (reinterpret_cast<uintptr_t>(W) & 15) || (int64_t)groups * N > 0x7fffffff)
     return (int)cudaErrorInvalidValue;
-  const Groups g{group_of_tile, num_tiles, N};
-  const GateAct act{1.f, 0.f, 0.f};
+  if (row_scale != nullptr && !gated) return (int)cudaErrorInvalidValue;
+  const Groups g{group_of_tile, num_tiles, N, row_scale};
+  const GateAct act{slope, limit, offset};
   const int w_rows = groups * N;
 #define GLLM_GROUPED(BN, OutT, GATED, ldo) \
   return umma_launch<BN, false, OutT, GATED>(X, W, (OutT*)out, rows, N, K, K, K, ldo, 1, nullptr, nullptr, 0, status, \

@@ -10,10 +10,14 @@
 //                `tile_m` rows (the last one filled up with -1), so that a tile of the products below reads ONE
 //                expert's weights; writes the pair of every row, the expert of every tile and the tile count.
 //   moe_gemm     out[pair] = A[row of pair] @ W[expert]^T over the tiles; `gated`: W holds gate and up rows and
-//                the result is silu(gate) * up, rounded to T; `act` 1 (experts without a gate): the square of
+//                the result is the gated activation of the two (GateAct: silu(gate) * up, or with a slope, clamps and
+//                an offset), rounded to T; `act` 1 (experts without a gate): the square of
 //                max(result, 0), rounded to T; otherwise the fp32 result itself.
 //   moe_combine  out[token] = sum over its slots, in slot order, of weight * result[pair] (+ a shared expert's
 //                result, times sigmoid(shared_gate[token]) when the shared expert has a gate), rounded to T.
+// A weight may instead multiply the expert's INPUT (W (w h) = w (W h)): moe_gemm (`row_scale`, one number per pair) and
+// the grouped tensor-core product (one per sorted row, filled in by moe_gather) multiply the fp32 accumulators by it
+// ahead of the activation, and moe_combine then adds without weights.
 // A pair's result does not depend on which other pairs share its tile or on the tile's place: every row is a dot
 // product over K in one fixed order.  Scores, choice, weights, accumulators and the combination are fp32.
 #include "common.cuh"
@@ -170,15 +174,16 @@ moe_align_kernel(const int* __restrict__ ids, int* __restrict__ sorted, int* __r
   }
 }
 
-// out[row_of_pair[p]] = x[p / top]: the tokens' rows in the order of the sorted pairs, for products that read
-// their rows in place (16 bytes a thread; width * sizeof(T) is a multiple of 16).
+// out[row_of_pair[p]] = x[p / top]: the tokens' rows in the order of the sorted pairs (and, with row_scale, the pairs'
+// weights in that order), for products that read their rows in place (16 bytes a thread; width * sizeof(T) is a multiple of 16).
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(const T* __restrict__ x, int64_t x_stride, const int* __restrict__ row_of_pair, T* __restrict__ out,
-                  int top, int width) {
+                  int top, int width, const float* __restrict__ weights, float* __restrict__ row_scale) {
   pdl_trigger();
   pdl_wait();
   const int p = blockIdx.x;
+  if (row_scale && threadIdx.x == 0) row_scale[row_of_pair[p]] = weights[p];
   const uint4* src = reinterpret_cast<const uint4*>(x + (int64_t)(p / top) * x_stride);
   uint4* dst = reinterpret_cast<uint4*>(out + (int64_t)row_of_pair[p] * width);
   const int n16 = width * (int)sizeof(T) / 16;
@@ -194,7 +199,7 @@ __global__ void __launch_bounds__(MG_THREADS)
 moe_gemm_kernel(const T* __restrict__ a, int64_t a_stride, int a_div, const T* __restrict__ w, int64_t w_expert_stride,
                 int64_t up_offset, const int* __restrict__ sorted, const int* __restrict__ tile_expert,
                 const int* __restrict__ num_tiles, T* __restrict__ out_t, float* __restrict__ out_f, int n_cols, int k,
-                int act) {
+                int act, const float* __restrict__ row_scale, GateAct gate) {
   __shared__ float As[MG_M][MG_K + 1];
   __shared__ float Bs[MG_N][MG_K + 1];
   __shared__ float Us[MG_N][MG_K + 1];
@@ -246,18 +251,23 @@ moe_gemm_kernel(const T* __restrict__ a, int64_t a_stride, int a_div, const T* _
   for (int i = 0; i < 2; ++i) {
     const int p = pairs[2 * ty + i];
     if (p < 0) continue;
+    const float rs = row_scale ? row_scale[p] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = col0 + tx + 16 * j;
       if (c >= n_cols) continue;
       if (gated) {
-        const float g = acc[i][j];
-        out_t[(int64_t)p * n_cols + c] = from_float<T>(g / (1.0f + expf(-g)) * acu[i][j]);
+        float g = acc[i][j] * rs, u = acu[i][j] * rs;
+        if (gate.limit > 0.f) {
+          g = fminf(g, gate.limit);
+          u = fminf(fmaxf(u, -gate.limit), gate.limit);
+        }
+        out_t[(int64_t)p * n_cols + c] = from_float<T>(g / (1.0f + expf(-gate.slope * g)) * (u + gate.offset));
       } else if (act == 1) {
-        const float r = fmaxf(acc[i][j], 0.f);
+        const float r = fmaxf(acc[i][j] * rs, 0.f);
         out_t[(int64_t)p * n_cols + c] = from_float<T>(r * r);
       } else {
-        out_f[(int64_t)p * n_cols + c] = acc[i][j];
+        out_f[(int64_t)p * n_cols + c] = acc[i][j] * rs;
       }
     }
   }
@@ -276,7 +286,7 @@ moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ weight
     float acc = 0.f;
     for (int s = 0; s < top; ++s) {
       const int64_t row = row_of_pair ? (int64_t)row_of_pair[t * top + s] : t * top + s;
-      acc = fmaf(weights[t * top + s], y[row * width + c], acc);
+      acc = fmaf(weights ? weights[t * top + s] : 1.f, y[row * width + c], acc);
     }
     if (shared) acc = fmaf(sg, to_float(shared[t * width + c]), acc);
     out[t * width + c] = from_float<T>(acc);
@@ -298,13 +308,14 @@ moe_relu_sq_kernel(const float* __restrict__ in, T* __restrict__ out, int64_t n)
 template <typename T>
 int moe_gemm_launch(const T* a, int64_t a_stride, int a_div, const T* w, int64_t w_expert_stride, int64_t up_offset,
                     const int* sorted, const int* tile_expert, const int* num_tiles, void* out, int max_tiles,
-                    int n_cols, int k, int tile_m, int act, cudaStream_t stream) {
+                    int n_cols, int k, int tile_m, int act, const float* row_scale, GateAct gate, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
   if (tile_m != MG_M || n_cols < 1 || k < 1 || a_div < 1 || act < 0 || act > 1) return (int)cudaErrorInvalidValue;
   const bool gated = up_offset != 0 || act == 1;
   return gllm_launch(moe_gemm_kernel<T>, dim3(max_tiles, (n_cols + MG_N - 1) / MG_N), dim3(MG_THREADS), 0, stream, a,
                      a_stride, a_div, w, w_expert_stride, up_offset, sorted, tile_expert, num_tiles,
-                     gated ? (T*)out : (T*)nullptr, gated ? (float*)nullptr : (float*)out, n_cols, k, act);
+                     gated ? (T*)out : (T*)nullptr, gated ? (float*)nullptr : (float*)out, n_cols, k, act, row_scale,
+                     gate);
 }
 }  // namespace
 
@@ -332,16 +343,19 @@ GLLM_API int gllm_moe_align(const int* ids, int* sorted, int* tile_expert, int* 
 
 GLLM_API int gllm_moe_gemm_f32(const float* a, int64_t a_stride, int a_div, const float* w, int64_t w_expert_stride,
                                int64_t up_offset, const int* sorted, const int* tile_expert, const int* num_tiles,
-                               void* out, int max_tiles, int n_cols, int k, int tile_m, int act, cudaStream_t stream) {
+                               void* out, int max_tiles, int n_cols, int k, int tile_m, int act,
+                               const float* row_scale, float slope, float limit, float offset, cudaStream_t stream) {
   return moe_gemm_launch<float>(a, a_stride, a_div, w, w_expert_stride, up_offset, sorted, tile_expert, num_tiles, out,
-                                max_tiles, n_cols, k, tile_m, act, stream);
+                                max_tiles, n_cols, k, tile_m, act, row_scale, GateAct{slope, limit, offset}, stream);
 }
 GLLM_API int gllm_moe_gemm_bf16(const __nv_bfloat16* a, int64_t a_stride, int a_div, const __nv_bfloat16* w,
                                 int64_t w_expert_stride, int64_t up_offset, const int* sorted, const int* tile_expert,
                                 const int* num_tiles, void* out, int max_tiles, int n_cols, int k, int tile_m,
-                                int act, cudaStream_t stream) {
+                                int act, const float* row_scale, float slope, float limit, float offset,
+                                cudaStream_t stream) {
   return moe_gemm_launch<__nv_bfloat16>(a, a_stride, a_div, w, w_expert_stride, up_offset, sorted, tile_expert,
-                                        num_tiles, out, max_tiles, n_cols, k, tile_m, act, stream);
+                                        num_tiles, out, max_tiles, n_cols, k, tile_m, act, row_scale,
+                                        GateAct{slope, limit, offset}, stream);
 }
 
 GLLM_API int gllm_moe_combine_f32(const float* y, const float* weights, const float* shared, float* out,
@@ -359,11 +373,13 @@ GLLM_API int gllm_moe_combine_bf16(const float* y, const float* weights, const _
                      row_of_pair, top, width, shared_gate, shared_gate_stride);
 }
 GLLM_API int gllm_moe_gather_bf16(const __nv_bfloat16* x, int64_t x_stride, const int* row_of_pair, __nv_bfloat16* out,
-                                  int n_pairs, int top, int width, cudaStream_t stream) {
+                                  int n_pairs, int top, int width, const float* weights, float* row_scale,
+                                  cudaStream_t stream) {
   if (n_pairs <= 0) return 0;
-  if (width % 8 || x_stride % 8 || top < 1 || (reinterpret_cast<uintptr_t>(x) & 15)) return (int)cudaErrorInvalidValue;
+  if (width % 8 || x_stride % 8 || top < 1 || (reinterpret_cast<uintptr_t>(x) & 15) || (row_scale && !weights))
+    return (int)cudaErrorInvalidValue;
   return gllm_launch(moe_gather_kernel<__nv_bfloat16>, dim3(n_pairs), dim3(256), 0, stream, x, x_stride, row_of_pair, out,
-                     top, width);
+                     top, width, weights, row_scale);
 }
 
 GLLM_API int gllm_moe_relu_sq_bf16(const float* in, __nv_bfloat16* out, int64_t n, cudaStream_t stream) {

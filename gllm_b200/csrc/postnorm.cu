@@ -5,6 +5,8 @@
 // (summed in ascending order and rounded to T, as the product would have); `extra` is a second fp32 stream
 // that is added as it is (the embedding output that a repeated stretch of layers takes in again).  With
 // `rows` only those rows are normed and resid stays untouched (the final norm at the wanted rows).
+// Without w nothing is normed on the way out: out[r] is the new resid[r] rounded to T (layers whose sublayers read the
+// residual itself).
 // Statistics, the normed value and the sums are fp32 whatever T is.
 #include "common.cuh"
 
@@ -103,8 +105,9 @@ postnorm_add_rmsnorm_kernel(const T* __restrict__ value, const float* __restrict
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v[e] += a[e];
     }
-    store_cols<VEC>(xs + c, v);
-    if (!rows) store_cols<VEC>(x + c, v);
+    if (w) store_cols<VEC>(xs + c, v);
+    else store_cols<VEC>(out + (int64_t)blockIdx.x * hidden + c, v);
+    if (!rows && (has_value || extra)) store_cols<VEC>(x + c, v);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ss2 = fmaf(v[e], v[e], ss2);
   }

@@ -108,7 +108,8 @@ class DecoderModel:
     # ------------------------------------------------------------------ cache
     def cache_requirements(self):
         """Per plan entry: (kv requirement | None, state requirement | None,
-        reads_cache_of | None)."""
+        reads_cache_of | None).  The state of an entry that reads another's cache is None unless its mixer keeps its
+        states itself (``Mixer.keeps_own_states``)."""
         out = []
         for entry in self.spec.plan:
             block = self.layers[entry.layer]
@@ -119,13 +120,20 @@ class DecoderModel:
             if extra:
                 own = () if state is None else (state,) if isinstance(state, StateRequirement) else tuple(state)
                 state = own + extra
+            if entry.reads_cache_of is not None:
+                if not (mixer is not None and mixer.keeps_own_states):
+                    state = None
+                owner_kv, owner_state, _ = out[entry.reads_cache_of]
+                if kv is not None and owner_kv is not None and kv != owner_kv:
+                    # the pages keep what every entry that attends over them needs
+                    out[entry.reads_cache_of] = (owner_kv.shared_with(kv), owner_state, None)
             out.append((kv, state, entry.reads_cache_of))
         return out
 
     def kernel_needs(self) -> dict:
         """Union of what the parts will ask of the kernel modules (``Part.kernel_needs``)."""
         needs: dict = {}
-        parts = [self.final_norm] + [p for block in self.layers for p in block.parts()]
+        parts = [self.final_norm] + [p for block in self.layers for p in [block] + block.parts()]
         for part in parts:
             for key, values in part.kernel_needs().items():
                 needs.setdefault(key, set()).update(values)

@@ -26,6 +26,7 @@ __all__ = [
     "scale_softcap",
     "scatter_int32",
     "add_rmsnorm",
+    "add_cast",
     "silu_mul",
     "rope_store",
     "linear",
@@ -135,6 +136,10 @@ _SIGNATURES = {
     "postnorm": {
         "gllm_postnorm_add_rmsnorm_{t}": [P, P, c_int, c_int64, P, c_float, P, P, P, c_float, P, P, c_int, c_int, P],
     },
+    "conv_qkv": {
+        "gllm_conv_qkv_{t}": [P, c_int64, P, c_int, c_int64, P, P, P, P, P, P, P, P, c_float, P, c_int, c_float, P, P,
+                              P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, P],
+    },
     "rope_norm": {
         "gllm_rope_norm_store_{t}": [P, P, c_int, c_int64, P, P, c_float, P, P, c_int, c_int, c_int, c_int, c_int,
                                      c_int, c_int, c_float, c_int, c_int, P, P],
@@ -148,10 +153,11 @@ _SIGNATURES = {
         "gllm_moe_route": [P, c_int64, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                            P],
         "gllm_moe_align": [P, P, P, P, P, c_int, c_int, c_int, c_int, P],
-        "gllm_moe_gemm_{t}": [P, c_int64, c_int, P, c_int64, c_int64, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P],
+        "gllm_moe_gemm_{t}": [P, c_int64, c_int, P, c_int64, c_int64, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P,
+                              c_float, c_float, c_float, P],
         "gllm_moe_combine_{t}": [P, P, P, P, P, c_int, c_int, c_int, P, c_int64, P],
         "gllm_moe_relu_sq_bf16": [P, P, c_int64, P],
-        "gllm_moe_gather_{t}": [P, c_int64, P, P, c_int, c_int, c_int, P],
+        "gllm_moe_gather_{t}": [P, c_int64, P, P, c_int, c_int, c_int, P, P, P],
     },
     "attention_simt": {
         "gllm_attention_simt_{t}": [P, c_int64, P, c_int64, P, P, c_int, P, P, c_int, c_int, c_int, c_int, c_int,
@@ -547,8 +553,16 @@ def add_rmsnorm(
     return out
 
 
+def add_cast(branch, resid: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """``resid += branch`` (fp32, in place; a ``Pending`` is normed first where it says so) and the sum rounded to
+    ``out_dtype``: what a sublayer reads that no norm precedes (``csrc/postnorm.cu``)."""
+    _cuda(resid, "resid", torch.float32)
+    return _pending_add_rmsnorm(Pending.of(branch), resid, None, 0.0, out_dtype, None, None)
+
+
 def _pending_add_rmsnorm(pending: Pending, resid, weight, eps, out_dtype, rows, out):
-    """``resid += rms(value) * post_weight + extra`` and the RMS norm of the sum (``csrc/postnorm.cu``)."""
+    """``resid += rms(value) * post_weight + extra`` and the RMS norm of the sum, or without ``weight`` the sum itself
+    (``csrc/postnorm.cu``)."""
     n_total, hidden = resid.numel() // resid.shape[-1], resid.shape[-1]
     value = pending.value
     parts_ptr, n_parts, part_stride = _parts_args(value)
@@ -577,7 +591,7 @@ def _pending_add_rmsnorm(pending: Pending, resid, weight, eps, out_dtype, rows, 
         _cuda(out, "out", out_dtype)
     f = _fn("postnorm", f"gllm_postnorm_add_rmsnorm_{_suffix(out_dtype)}")
     _check(f(_ptr(value), parts_ptr, n_parts, part_stride, _ptr(pending.post_weight), pending.post_eps,
-             _ptr(pending.extra), resid.data_ptr(), weight.data_ptr(), float(eps), out.data_ptr(), _ptr(rows), n_rows,
+             _ptr(pending.extra), resid.data_ptr(), _ptr(weight), float(eps), out.data_ptr(), _ptr(rows), n_rows,
              hidden, _stream()), "postnorm_add_rmsnorm")
     return out
 
@@ -956,11 +970,13 @@ def paged_attention(
     window: int | None = None,
     batch=None,
     out: torch.Tensor | None = None,
+    chunk: int | None = None,
 ) -> torch.Tensor:
-    """Causal attention of every token of the batch over its request's cache.
+    """Causal attention of every token of the batch over its request's cache: over all keys, the last ``window``, or
+    (``chunk``) those of the query's own chunk of ``chunk`` positions, counted from the sequence's start.
 
     ``qkv`` is ``[n, (heads + 2*kv_heads) * head_dim]`` with rotated queries in
-    its first ``heads * head_dim`` columns; the keys and values of the batch's
+    its first ``heads * head_dim`` columns, or those columns alone; the keys and values of the batch's
     own tokens are already in ``cache_layer``.  ``token_row[i]`` is the row of
     ``block_table`` that token ``i``'s request uses.  ``batch`` optionally
     carries per-request metadata that the tensor-core kernels need.
@@ -978,13 +994,17 @@ def paged_attention(
     if num_heads % hkv:
         raise ValueError("the number of query heads must be a multiple of the number of kv heads")
     n = qkv.shape[0]
-    if qkv.shape[1] != (num_heads + 2 * hkv) * d:
-        raise ValueError("qkv width does not equal (heads + 2*kv_heads) * head_dim")
+    if qkv.shape[1] not in ((num_heads + 2 * hkv) * d, num_heads * d):
+        raise ValueError("qkv width equals neither (heads + 2*kv_heads) * head_dim nor heads * head_dim")
     if block_table.stride(1) != 1:
         raise ValueError("block_table rows must be contiguous")
     if out is None:
         out = torch.empty((n, num_heads * d), dtype=qkv.dtype, device=qkv.device)
     win = int(window) if window else 0
+    if chunk:
+        if win:
+            raise ValueError("a layer has a window or chunks, not both")
+        win = -int(chunk)                 # the kernels' way of saying it (first_visible_key in csrc/common.cuh)
     if qkv.dtype == torch.bfloat16:
         from gllm_b200.ops import attention_bf16
 

@@ -152,9 +152,24 @@ def supports(head_dim: int, block_size: int) -> bool:
     return head_dim in _DECODE_HEAD_DIMS and (block_size * head_dim) % 8 == 0
 
 
-def decode_scratch_elems(num_queries: int, num_heads: int, head_dim: int, max_seq_len: int) -> tuple[int, int, int]:
+def visible_spans(max_seq_len: int, span: int, window: int) -> int:
+    """How many spans of ``span`` keys (aligned to multiples of ``span``) the keys one query sees can touch; ``window``
+    as the kernels take it (> 0 a window, < 0 chunks of ``-window`` positions, 0 everything)."""
+    total = max(1, -(-max_seq_len // span))
+    if window == 0:
+        return total
+    size = abs(window)
+    if window < 0 and size % span == 0:
+        return min(total, size // span)
+    if window < 0 and span % size == 0:
+        return 1
+    return min(total, -(-(size - 1) // span) + 1)
+
+
+def decode_scratch_elems(num_queries: int, num_heads: int, head_dim: int, max_seq_len: int,
+                         window: int = 0) -> tuple[int, int, int]:
     """(num_chunks, floats of partial outputs, floats of partial max/sum)."""
-    chunks = max(1, -(-max_seq_len // decode_chunk(head_dim)))
+    chunks = visible_spans(max_seq_len, decode_chunk(head_dim), window)
     return chunks, num_queries * num_heads * chunks * head_dim, num_queries * num_heads * chunks * 2
 
 
@@ -171,14 +186,14 @@ def decode_attention(q, q_stride, cache_layer, block_table, positions, token_row
     if kernel == "stream" and not parts:
         raise ValueError(f"the stream decode kernel does not take {num_heads}/{hkv} heads of {d} with pages of "
                          f"{block_size}")
-    spans = max(1, -(-max_seq_len // STREAM_SPAN))
+    spans = visible_spans(max_seq_len, STREAM_SPAN, int(window))
     use_stream = bool(parts) and (kernel == "stream" or n * spans >= STREAM_MIN_ITEMS)
     if use_stream:
         chunks = spans
         n_o, n_ml = n * num_heads * spans * parts * d, n * num_heads * spans * parts * 2
         fn, name = _decode_stream_fn()[0], "attention_decode_stream"
     else:
-        chunks, n_o, n_ml = decode_scratch_elems(n, num_heads, d, max_seq_len)
+        chunks, n_o, n_ml = decode_scratch_elems(n, num_heads, d, max_seq_len, int(window))
         fn, name = _decode_fn()[0], "attention_decode_bf16"
     if workspace is not None:
         part_o = workspace.get("attention_decode_partial_out", n_o, torch.float32)

@@ -56,6 +56,7 @@ MODULES = {
     "attention_latent_mma": "attention_latent_mma.cu",
     "postnorm": "postnorm.cu",
     "rope_norm": "rope_norm.cu",
+    "conv_qkv": "conv_qkv.cu",
     "delta_rule": "delta_rule.cu",
     "moe": "moe.cu",
     "dyt_norm": "dyt_norm.cu",

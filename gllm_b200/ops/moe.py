@@ -9,6 +9,7 @@ import torch
 from gllm_b200.ops import _check, _cuda, _fn, _ptr, _stream, _suffix
 
 TILE_ROWS = 16        # rows of one tile of the expert products: an expert's pairs are padded to a multiple of it
+PLAIN_GATE = (1.0, 0.0, 0.0)    # slope, limit, offset of a gated expert's activation: silu(gate) * up
 TENSOR_CORE_TILE_ROWS = 128     # the same for the tcgen05 products (the rows of one accumulator tile)
 
 
@@ -58,15 +59,23 @@ def align(ids: torch.Tensor, experts: int, tile_rows: int = TILE_ROWS, want_rows
     return sorted_pairs, tile_expert, num_tiles
 
 
-def gather_rows(x: torch.Tensor, top: int, row_of_pair: torch.Tensor, rows: int) -> torch.Tensor:
+def gather_rows(x: torch.Tensor, top: int, row_of_pair: torch.Tensor, rows: int, weights: torch.Tensor | None = None):
     """``out[row_of_pair[p]] = x[p // top]`` (bf16, ``[rows, width]``): the tokens' rows in the order of the sorted
-    pairs.  Rows that no pair owns are left as they are: the products' rows do not mix, and nobody reads theirs."""
+    pairs; with ``weights`` (fp32, one per pair) also ``[rows]`` of those in the same order: ``(out, row_scale)``.  Rows
+    that no pair owns are left as they are: the products' rows do not mix, and nobody reads theirs."""
     _cuda(x, "x", torch.bfloat16, contiguous=False)
     _cuda(row_of_pair, "row_of_pair", torch.int32)
     out = torch.empty((rows, x.shape[1]), dtype=x.dtype, device=x.device)
+    row_scale = None
+    if weights is not None:
+        _cuda(weights, "weights", torch.float32)
+        if weights.numel() != row_of_pair.numel():
+            raise ValueError("one weight per (token, slot) pair is needed")
+        row_scale = torch.empty(rows, dtype=torch.float32, device=x.device)
     _check(_fn("moe", "gllm_moe_gather_bf16")(x.data_ptr(), x.stride(0), row_of_pair.data_ptr(), out.data_ptr(),
-                                              row_of_pair.numel(), int(top), x.shape[1], _stream()), "moe_gather")
-    return out
+                                              row_of_pair.numel(), int(top), x.shape[1], _ptr(weights), _ptr(row_scale),
+                                              _stream()), "moe_gather")
+    return out if weights is None else (out, row_scale)
 
 
 def tensor_cores_take(dtype: torch.dtype, width: int, ff: int, gated: bool = True) -> bool:
@@ -76,10 +85,12 @@ def tensor_cores_take(dtype: torch.dtype, width: int, ff: int, gated: bool = Tru
 
 
 def expert_product(a: torch.Tensor, rows_per_input: int, weight: torch.Tensor, plan, n_pairs: int, gated: bool,
-                   relu_squared: bool = False):
+                   relu_squared: bool = False, act: tuple = PLAIN_GATE, row_scale: torch.Tensor | None = None):
     """``out[pair] = a[pair // rows_per_input] @ weight[expert of pair].T`` for the pairs of ``plan`` (what
     ``align`` returned).  ``weight [experts, rows, k]``; ``gated``: its rows are gate rows then up rows and the
-    result is ``silu(gate) * up`` in the activation type ``[n_pairs, rows / 2]``; ``relu_squared`` (experts without a
+    result is ``silu(gate) * up`` (or what ``act``, the slope, limit and offset of ``ops.linear_gated``, says) in the
+    activation type ``[n_pairs, rows / 2]``; ``row_scale`` (fp32, one number per pair): the products are multiplied by
+    it, ahead of the activation; ``relu_squared`` (experts without a
     gate): ``max(result, 0) ** 2`` in the activation type ``[n_pairs, rows]``; otherwise fp32 ``[n_pairs, rows]``."""
     _cuda(a, "a", contiguous=False)
     _cuda(weight, "weight", a.dtype)
@@ -94,13 +105,16 @@ def expert_product(a: torch.Tensor, rows_per_input: int, weight: torch.Tensor, p
     f = _fn("moe", f"gllm_moe_gemm_{_suffix(a.dtype)}")
     _check(f(a.data_ptr(), a.stride(0), int(rows_per_input), weight.data_ptr(), weight.stride(0),
              n_cols * k if gated else 0, sorted_pairs.data_ptr(), tile_expert.data_ptr(), num_tiles.data_ptr(),
-             out.data_ptr(), tile_expert.numel(), n_cols, k, TILE_ROWS, int(relu_squared), _stream()), "moe_gemm")
+             out.data_ptr(), tile_expert.numel(), n_cols, k, TILE_ROWS, int(relu_squared), _ptr(row_scale), *act, _stream()),
+           "moe_gemm")
     return out
 
 
 def combine(y: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None, out_dtype: torch.dtype,
-            row_of_pair: torch.Tensor | None = None, shared_gate: torch.Tensor | None = None) -> torch.Tensor:
-    """``out[t] = sum_s weights[t, s] * y[t * top + s] (+ shared[t])``, summed in slot order in fp32; with
+            row_of_pair: torch.Tensor | None = None, shared_gate: torch.Tensor | None = None,
+            weighted: bool = True) -> torch.Tensor:
+    """``out[t] = sum_s weights[t, s] * y[t * top + s] (+ shared[t])``, summed in slot order in fp32 (``weighted``
+    False: without the weights, which the experts' inputs had); with
     ``row_of_pair`` the pair's result is row ``row_of_pair[t * top + s]`` of ``y``; with ``shared_gate`` (fp32, one
     logit per token; may be a column of a wider matrix) the shared result is multiplied by its sigmoid."""
     _cuda(y, "y", torch.float32)
@@ -122,7 +136,8 @@ def combine(y: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None,
             raise ValueError("the shared expert's gate is one logit per token")
         gate_stride = shared_gate.stride(0)
     out = torch.empty((n, width), dtype=out_dtype, device=y.device)
-    _check(_fn("moe", f"gllm_moe_combine_{_suffix(out_dtype)}")(y.data_ptr(), weights.data_ptr(), _ptr(shared),
+    _check(_fn("moe", f"gllm_moe_combine_{_suffix(out_dtype)}")(y.data_ptr(),
+                                                               weights.data_ptr() if weighted else None, _ptr(shared),
                                                                out.data_ptr(), _ptr(row_of_pair), n, top, width,
                                                                _ptr(shared_gate), gate_stride, _stream()), "moe_combine")
     return out
@@ -139,27 +154,38 @@ def relu_squared_rows(x: torch.Tensor) -> torch.Tensor:
 
 def apply_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                   w_down: torch.Tensor, shared: torch.Tensor | None, tensor_cores: bool, gated: bool = True,
-                  shared_gate: torch.Tensor | None = None) -> torch.Tensor:
+                  shared_gate: torch.Tensor | None = None, act: tuple = PLAIN_GATE,
+                  weight_on_input: bool = False) -> torch.Tensor:
     """``out[t] = sum_s weights[t, s] * expert_{ids[t, s]}(x[t]) (+ shared[t])`` with ``expert_e(x) = w_down[e]
     (silu(gate) * up)``.  ``tensor_cores``: ``w_gate_up [experts, 2 * ff, width]`` is stacked per expert by
     ``interleave_gate_up``; the tokens' rows are copied into the order of the sorted pairs, both products read and
     write rows in that order on the tcgen05 kernel, and the weighted sum looks every pair's row up.  Otherwise
     ``w_gate_up`` holds an expert's gate rows, then its up rows, and the CUDA-core kernel runs.  ``gated`` False:
     experts without a gate, ``expert_e(x) = w_down[e] relu(w_up[e] x)^2`` with ``w_gate_up [experts, ff, width]`` the
-    up weights.  ``shared_gate``: see ``combine``."""
+    up weights.  ``shared_gate``: see ``combine``.  ``act``: the slope, limit and offset of the gated activation.
+    ``weight_on_input``: ``out[t] = sum_s expert(weights[t, s] * x[t])`` instead; the weight is applied to the first
+    product's fp32 sums, which is the same and spares a rounding."""
     experts, (_, top), pairs = w_gate_up.shape[0], ids.shape, ids.numel()
     if not tensor_cores:
         plan = align(ids, experts)
-        hidden = expert_product(x, top, w_gate_up, plan, pairs, gated=gated, relu_squared=not gated)
+        hidden = expert_product(x, top, w_gate_up, plan, pairs, gated=gated, relu_squared=not gated, act=act,
+                                row_scale=weights if weight_on_input else None)
         y = expert_product(hidden, 1, w_down, plan, pairs, gated=False)
-        return combine(y, weights, shared, x.dtype, shared_gate=shared_gate)
+        return combine(y, weights, shared, x.dtype, shared_gate=shared_gate, weighted=not weight_on_input)
     from gllm_b200.ops import gemm_bf16
 
     _, tile_expert, num_tiles, row_of_pair = align(ids, experts, TENSOR_CORE_TILE_ROWS, want_rows=True)
     wide = pairs > 2048
-    xs = gather_rows(x, top, row_of_pair, tile_expert.numel() * TENSOR_CORE_TILE_ROWS)
-    hidden = gemm_bf16.linear_grouped(xs, w_gate_up, tile_expert, num_tiles, gated=gated, wide=wide)
+    rows, row_scale = tile_expert.numel() * TENSOR_CORE_TILE_ROWS, None
+    if weight_on_input:
+        if not gated:
+            raise ValueError("weights on the input of the tensor-core products are for gated experts")
+        xs, row_scale = gather_rows(x, top, row_of_pair, rows, weights)
+    else:
+        xs = gather_rows(x, top, row_of_pair, rows)
+    hidden = gemm_bf16.linear_grouped(xs, w_gate_up, tile_expert, num_tiles, gated=gated, wide=wide, act=act,
+                                      row_scale=row_scale)
     if not gated:
         hidden = relu_squared_rows(hidden)
     y = gemm_bf16.linear_grouped(hidden, w_down, tile_expert, num_tiles, gated=False, wide=wide)
-    return combine(y, weights, shared, x.dtype, row_of_pair, shared_gate=shared_gate)
+    return combine(y, weights, shared, x.dtype, row_of_pair, shared_gate=shared_gate, weighted=not weight_on_input)

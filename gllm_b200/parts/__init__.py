@@ -32,8 +32,8 @@ from gllm_b200.parts.base import (
     register_position_encoding,
 )
 from gllm_b200.parts import (  # noqa: F401  (register the built-in kinds)
-    attention, block, delta_rule, depth, differential_attention, distance_attention, experts, hyper, latent_attention,
-    mamba, matrix_memory, mlp, norm, parallel, rotary, sigmoid_attention,
+    attention, block, conv_attention, delta_rule, depth, differential_attention, distance_attention, experts, hyper,
+    latent_attention, mamba, matrix_memory, mlp, norm, parallel, rotary, sigmoid_attention,
 )
 
 __all__ = [

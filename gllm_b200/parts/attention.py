@@ -26,6 +26,21 @@ from gllm_b200.parts.base import (
 )
 
 
+# head widths the tensor-core attention kernels are built for
+KERNEL_WIDTHS = (32, 64, 128)
+
+
+def stored_head_width(dk: int, dv: int) -> int:
+    """The width that query and key heads of ``dk`` and value heads of ``dv`` columns are stored at when they are padded
+    to one: the next the tensor-core kernels take, beyond those the larger of the two rounded up to 8."""
+    widest = max(dk, dv)
+    fitting = [w for w in KERNEL_WIDTHS if w >= widest]
+    width = fitting[0] if fitting else -(-widest // 8) * 8
+    if not 0 < min(dk, dv) or width > 256:
+        raise ValueError("the attention kernels take head sizes up to 256")
+    return width
+
+
 @register_mixer("attention")
 class Attention(Mixer):
     graph_safe_portions = True
@@ -89,20 +104,12 @@ class Attention(Mixer):
         self.w_q_norm: torch.Tensor | None = None
         self.w_k_norm: torch.Tensor | None = None
 
-    # head widths the tensor-core attention kernels are built for
-    KERNEL_WIDTHS = (32, 64, 128)
-
     def _cache_dim(self) -> int:
-        widest = max(self.head_dim, self.value_dim)
         if not self.pad_heads:
             if self.value_dim != self.head_dim:
                 raise ValueError("key and value heads of different widths need pad_heads")
             return self.head_dim
-        fitting = [w for w in self.KERNEL_WIDTHS if w >= widest]
-        width = fitting[0] if fitting else -(-widest // 8) * 8
-        if width > 256:
-            raise ValueError("the attention kernels take head sizes up to 256")
-        return width
+        return stored_head_width(self.head_dim, self.value_dim)
 
     def kv_requirement(self):
         return KVPageRequirement.keys_and_values(self.num_kv_heads, self.cache_dim, self.window)

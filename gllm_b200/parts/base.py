@@ -64,10 +64,16 @@ class KVPageRequirement:
     window: int | None = None
     # ... and, for as long as the request lives, the positions below this one
     keep_first: int = 0
+    # (c, ..): the sequence is cut into chunks of c positions, counted from position 0, and a token at position p
+    # needs those of its own chunk, p // c * c on (several sizes when layers with chunks of their own share the pages:
+    # the earliest position counts, also against the window's)
+    chunks: tuple[int, ...] = ()
 
     def __post_init__(self):
         if not self.tensors or any(len(t) != 2 or t[0] <= 0 or t[1] <= 0 for t in self.tensors):
             raise ValueError("a page requirement names at least one (heads, width) tensor of positive sizes")
+        if any(c <= 0 for c in self.chunks):
+            raise ValueError("chunks have a positive number of positions")
 
     @classmethod
     def keys_and_values(cls, num_kv_heads: int, head_dim: int, window: int | None = None) -> "KVPageRequirement":
@@ -77,6 +83,28 @@ class KVPageRequirement:
     @property
     def elements_per_token(self) -> int:
         return sum(h * w for h, w in self.tensors)
+
+    @property
+    def bounded(self) -> bool:
+        """Whether later tokens stop needing earlier positions at all."""
+        return self.window is not None or bool(self.chunks)
+
+    def first_needed(self, position: int) -> int:
+        """The first position (those of ``keep_first`` aside) that tokens at ``position`` and later still need."""
+        starts = [position // c * c for c in self.chunks]
+        if self.window is not None:
+            starts.append(max(0, position - self.window + 1))
+        return min(starts, default=0)
+
+    def shared_with(self, reader: "KVPageRequirement") -> "KVPageRequirement":
+        """What pages have to keep that a second entry with the requirement ``reader`` attends over as well."""
+        if reader.tensors != self.tensors:
+            raise ValueError("an entry reads the pages of another whose heads or widths differ from its own")
+        if not (self.bounded and reader.bounded):
+            return KVPageRequirement(self.tensors)
+        windows = [w for w in (self.window, reader.window) if w is not None]
+        return KVPageRequirement(self.tensors, max(windows, default=None), max(self.keep_first, reader.keep_first),
+                                 tuple(sorted(set(self.chunks) | set(reader.chunks))))
 
 
 @dataclass(frozen=True)
@@ -233,6 +261,10 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    # True: in a plan entry that reads another entry's pages the mixer still keeps its states itself (a convolution
+    # over its own queries); False: it then works on the states of the entry it reads.
+    keeps_own_states = False
+
     def kv_requirement(self) -> KVPageRequirement | None:
         return None
 

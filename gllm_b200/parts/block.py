@@ -55,6 +55,30 @@ class SharedNormBlock(Block):
         return out, resid
 
 
+@register_block("result_only_norm")
+class ResultOnlyNormBlock(Block):
+    """A norm on each sublayer's result and none before it: ``x += norm_a(mixer(x)); x += norm_b(ff(x))``; the
+    sublayers read the residual itself, rounded to the compute type (a factor on what is added is the norm's
+    ``multiplier``).  A sublayer's result travels on as ``ops.Pending``; the next sublayer's input kernel
+    (``ops.add_cast``) norms it, adds it and rounds in one pass.  A layer may have no feed-forward."""
+
+    graph_safe_portions = True
+    part_kinds = {"mixer": "mixer", "mixer_norm": "norm", "feed_forward": "feed_forward", "feed_forward_norm": "norm"}
+    optional_parts = frozenset({"feed_forward", "feed_forward_norm"})
+
+    def kernel_needs(self):
+        return {"modules": {"postnorm"}}
+
+    def forward(self, branch, resid, ctx, cache):
+        ctx.residual_sink = None
+        x = ops.add_cast(None if branch is ops.ADDED else branch, resid, ctx.dtype)
+        out = self.mixer_norm.pending(self.mixer.forward(x, ctx, cache))
+        if self.feed_forward is not None:
+            x = ops.add_cast(out, resid, ctx.dtype)
+            out = self.feed_forward_norm.pending(self.feed_forward.forward(x, ctx))
+        return out, resid
+
+
 @register_block("sandwich")
 class SandwichBlock(Block):
     """A norm before and a norm after each sublayer: ``x += post_a(mixer(pre_a(x))); x += post_b(ff(pre_b(x)))``.
@@ -67,6 +91,9 @@ class SandwichBlock(Block):
     part_kinds = {"mixer_norm": "norm", "mixer": "mixer", "mixer_post_norm": "norm",
                   "feed_forward_norm": "norm", "feed_forward": "feed_forward", "feed_forward_post_norm": "norm"}
     optional_parts = frozenset({"feed_forward_norm", "feed_forward", "feed_forward_post_norm"})
+
+    def kernel_needs(self):
+        return {"modules": {"postnorm"}}
 
     def forward(self, branch, resid, ctx, cache):
         ctx.residual_sink = None

@@ -14,7 +14,10 @@ Options for other designs: ``score`` "softmax" (scores are the softmax of the lo
 ``group_score`` "max" (a group's score is its largest choice score); ``renormalize_eps`` (added to the sum the
 weights are divided by); ``scale`` (the weights are multiplied by it last); ``expert`` "relu_squared": experts
 without a gate, ``down(max(up(x), 0) ** 2)``; ``shared_gate``: the shared expert's result is multiplied by
-``sigmoid(w_sg . x)``, one number per token (its row rides on the router's product).
+``sigmoid(w_sg . x)``, one number per token (its row rides on the router's product); ``gate_slope``, ``gate_limit`` and
+``up_offset``: the gated activation is ``g * sigmoid(slope * g) * (u + offset)`` of ``g = min(gate, limit)`` and ``u =
+clamp(up, -limit, limit)``; ``weight_on_input``: a weight multiplies what its expert reads instead of what it returns,
+``sum_e expert_e(s_e * x)``.
 """
 
 from __future__ import annotations
@@ -34,7 +37,8 @@ class RoutedExperts(FeedForward):
                  groups: int | None = None, groups_kept: int | None = None, score: str = "sigmoid",
                  renormalize: bool = False, correction: bool = False, shared=None, group_score: str = "top2",
                  renormalize_eps: float = 0.0, scale: float = 1.0, expert: str = "gated_silu",
-                 shared_gate: bool = False):
+                 shared_gate: bool = False, gate_slope: float = 1.0, gate_limit: float | None = None,
+                 up_offset: float = 0.0, weight_on_input: bool = False):
         """``names``: ``router``, ``correction`` (with ``correction``), ``shared_gate`` (with ``shared_gate``) and
         ``expert``, a pattern with ``{index}`` and ``{part}`` (gate | up | down).  ``shared``: the PartSpec of a
         feed-forward that runs for every token."""
@@ -47,6 +51,12 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"unknown expert form {expert!r}; known: ['gated_silu', 'relu_squared']")
         if shared_gate and shared is None:
             raise ValueError("a gate of the shared expert needs a shared expert")
+        if gate_limit is not None and not gate_limit > 0:
+            raise ValueError("the limit of the gate and up products is positive")
+        if expert != "gated_silu" and (weight_on_input or gate_limit is not None or gate_slope != 1.0 or up_offset != 0.0):
+            raise ValueError("the activation's constants and weights on the input are for gated experts")
+        self.act = (float(gate_slope), float(gate_limit or 0.0), float(up_offset))
+        self.weight_on_input = bool(weight_on_input)
         self.score, self.group_score, self.gated = score, group_score, expert == "gated_silu"
         self.renormalize_eps, self.scale, self.has_shared_gate = float(renormalize_eps), float(scale), bool(shared_gate)
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
@@ -121,4 +131,4 @@ class RoutedExperts(FeedForward):
             shared = ops.as_tensor(self.shared.forward(x, ctx))
             ctx.residual_sink = sink
         return moe.apply_experts(x, ids, weights, self.w_gate_up, self.w_down, shared, self.tensor_cores,
-                                 gated=self.gated, shared_gate=gate)
+                                 gated=self.gated, shared_gate=gate, act=self.act, weight_on_input=self.weight_on_input)

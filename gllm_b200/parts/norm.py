@@ -19,8 +19,12 @@ from gllm_b200.parts.base import Norm, TensorExpectation, register_norm
 class RMSNorm(Norm):
     graph_safe_portions = True
 
-    def __init__(self, names, size: int, eps: float, unit_offset: bool = False):
+    def __init__(self, names, size: int, eps: float, unit_offset: bool = False, multiplier: float = 1.0):
+        """``multiplier``: a constant factor on the normed rows (held in the weight)."""
         super().__init__(names)
+        self.multiplier = float(multiplier)
+        if unit_offset and self.multiplier != 1.0:
+            raise ValueError("a norm whose weight is stored around zero takes no multiplier")
         self.size = int(size)
         self.eps = float(eps)
         # True: the stored weight is an offset from one, y = x_hat * (1 + w)
@@ -32,6 +36,8 @@ class RMSNorm(Norm):
 
     def load(self, get, dtype, device):
         self.weight = get(self.names["weight"], "vector")
+        if self.multiplier != 1.0:
+            self.weight = self.weight * self.multiplier
 
     def depth_pending(self, value, streams=None, count: int = 0, depth_weight=None):
         """``value`` (a sublayer's result, possibly ``ops.Biased``) as an ``ops.DepthPending`` with this norm's weight,
