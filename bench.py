@@ -613,8 +613,25 @@ def vonedra_raw(sz: dict) -> dict:
             "torch_dtype": "bfloat16"}
 
 
+def pifelix_raw(sz: dict) -> dict:
+    """``layers`` layers of attention in chunks of 1,024 tokens (4 taps, scaled rotation over the whole head), the last
+    third reading the keys and values of the layer before them; routed experts everywhere (16 experts of ff/4, 4 per
+    token: as many active feed-forward weights per token as the dense layers of the Llama)."""
+    mixer = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": sz["head_dim"], "vdim": sz["head_dim"],
+             "scale": sz["head_dim"] ** -0.5, "conv": 4, "mask": {"size": 1024},
+             "rot": {"base": 10000.0, "dims": sz["head_dim"],
+                     "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}
+    routed = {"kind": "moe", "expert": {"ff": sz["ff"] // 4, "limit": 7.0}, "router": {"experts": 16, "top": 4}}
+    own = sz["layers"] - sz["layers"] // 3
+    return {"architecture": "Pifelix", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": 8.0}, "residual_mult": 0.5,
+            "layers": [{"type": "attention", "mixer": mixer if i < own else dict(mixer, kv_from=own - 1), "mlp": routed}
+                       for i in range(sz["layers"])],
+            "torch_dtype": "bfloat16"}
+
+
 DESIGNS = {"guvetar": guvetar_raw, "rulunex": rulunex_raw, "mifidra": mifidra_raw, "sazisun": sazisun_raw,
-           "vonedra": vonedra_raw}
+           "vonedra": vonedra_raw, "pifelix": pifelix_raw}
 
 
 def llama_raw(sz: dict) -> dict:

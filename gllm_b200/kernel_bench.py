@@ -50,7 +50,8 @@ def _paged_cache(batch, context, hkv, d, block_size, extra_tokens=0, sequential=
 
 
 def attention_decode(batch=64, context=2048, hq=32, hkv=8, d=64, block_size=16, iters=5, peaks=None, sequential=0,
-                     stream=1):
+                     stream=1, chunk=0):
+    """Single tokens over ``context`` cached ones, or (``chunk``) over those of the last token's own chunk."""
     from gllm_b200.ops import attention_bf16
 
     pool, table = _paged_cache(batch, context, hkv, d, block_size, sequential=sequential)
@@ -71,17 +72,19 @@ def attention_decode(batch=64, context=2048, hq=32, hkv=8, d=64, block_size=16, 
 
     ws = _WS()
     fn = lambda: attention_bf16.decode_attention(qkv, qkv.shape[1], pool, table, positions, rows, hq,
-                                                 1.0 / math.sqrt(d), 0, context, ws, out,
+                                                 1.0 / math.sqrt(d), -chunk, context, ws, out,
                                                  kernel="stream" if stream else "split")
     us = _time(fn, iters, flush)
-    nbytes = batch * context * 2 * hkv * d * 2
+    keys = (context - 1) % chunk + 1 if chunk else context
+    nbytes = batch * keys * 2 * hkv * d * 2
     gbs = nbytes / us / 1e3
     return {"kernel": "attention_decode (stream + merge)" if stream else "attention_decode (split + merge)", "us": round(us, 2), "bytes": nbytes,
             "achieved_gbs": round(gbs, 1), "frac_of_hbm_peak": round(gbs / peaks["hbm_gbs"], 4),
-            "shape": dict(batch=batch, context=context, heads=hq, kv_heads=hkv, head_dim=d, block_size=block_size)}
+            "shape": dict(batch=batch, context=context, heads=hq, kv_heads=hkv, head_dim=d, block_size=block_size, chunk=chunk)}
 
 
-def attention_prefill(tokens=2048, context=0, hq=32, hkv=8, d=64, block_size=16, iters=5, peaks=None, tmem=1):
+def attention_prefill(tokens=2048, context=0, hq=32, hkv=8, d=64, block_size=16, iters=5, peaks=None, tmem=1,
+                      chunk=0):
     from gllm_b200.ops import attention_bf16
 
     pool, table = _paged_cache(1, context + tokens, hkv, d, block_size)
@@ -92,13 +95,15 @@ def attention_prefill(tokens=2048, context=0, hq=32, hkv=8, d=64, block_size=16,
     out = torch.empty(tokens, hq * d, dtype=torch.bfloat16, device="cuda")
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
     kernel = attention_bf16.prefill_attention_tmem if tmem else attention_bf16.prefill_attention
-    fn = lambda: kernel(qkv, qkv.shape[1], pool, table, cu, ctx, slots, 1, tokens, hq, 1.0 / math.sqrt(d), 0, out)
+    fn = lambda: kernel(qkv, qkv.shape[1], pool, table, cu, ctx, slots, 1, tokens, hq, 1.0 / math.sqrt(d), -chunk, out)
     us = _time(fn, iters, flush)
-    flops = 4.0 * d * hq * (tokens * context + tokens * (tokens + 1) / 2)
+    pairs = (sum(p % chunk + 1 for p in range(context, context + tokens)) if chunk
+             else tokens * context + tokens * (tokens + 1) / 2)
+    flops = 4.0 * d * hq * pairs
     tf = flops / us / 1e6
     return {"kernel": "attention_prefill (tcgen05)" if tmem else "attention_prefill (mma.sync)", "us": round(us, 2), "flops": flops, "achieved_tflops": round(tf, 1),
             "frac_of_bf16_peak": round(tf / peaks["bf16_tflops"], 4),
-            "shape": dict(tokens=tokens, context=context, heads=hq, kv_heads=hkv, head_dim=d, block_size=block_size)}
+            "shape": dict(tokens=tokens, context=context, heads=hq, kv_heads=hkv, head_dim=d, block_size=block_size, chunk=chunk)}
 
 
 def linear(m=8, n=16384, k=2048, iters=5, peaks=None, out_fp32=False, gated=0, split=0, acc=0):
@@ -189,10 +194,11 @@ def decode_step(batch=8, context=2048, layers=2, iters=3, peaks=None):
     return {"kernel": "decode_step (no graph)", "us": round(us, 2), "shape": dict(batch=batch, context=context, layers=layers)}
 
 
-def add_rmsnorm(rows=8, hidden=2048, splits=8, post=0, iters=5, peaks=None):
+def add_rmsnorm(rows=8, hidden=2048, splits=8, post=0, cast=0, iters=5, peaks=None):
     """resid += (sum of ``splits`` fp32 partial products, 0: a summed bf16 branch), then RMSNorm: the
     kernel between two products of a layer.  ``post``: the branch is RMS-normed with a weight of its own
-    before it is added (the norm after a sublayer of a layer that norms both sides of it)."""
+    before it is added (the norm after a sublayer of a layer that norms both sides of it).  ``cast`` (with ``post``):
+    the new residual is rounded, not normed, on the way out."""
     from gllm_b200 import ops
 
     resid = torch.randn(rows, hidden, device="cuda")
@@ -203,10 +209,13 @@ def add_rmsnorm(rows=8, hidden=2048, splits=8, post=0, iters=5, peaks=None):
         branch = ops.Pending(branch, torch.ones(hidden, device="cuda"), 1e-5)
     out = torch.empty(rows, hidden, dtype=torch.bfloat16, device="cuda")
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
-    us = _time(lambda: ops.add_rmsnorm(branch, resid, weight, 1e-5, torch.bfloat16, out=out), iters, flush)
+    if cast:
+        us = _time(lambda: ops.add_cast(branch, resid, torch.bfloat16), iters, flush)
+    else:
+        us = _time(lambda: ops.add_rmsnorm(branch, resid, weight, 1e-5, torch.bfloat16, out=out), iters, flush)
     nbytes = rows * hidden * ((4 * splits if splits else 2) + 4 + 4 + 2) + hidden * 4 * (2 if post else 1)
     gbs = nbytes / us / 1e3
-    return {"kernel": "add_rmsnorm (normed branch)" if post else "add_rmsnorm", "us": round(us, 2), "bytes": nbytes,
+    return {"kernel": "add_cast (normed branch)" if cast else "add_rmsnorm (normed branch)" if post else "add_rmsnorm", "us": round(us, 2), "bytes": nbytes,
             "achieved_gbs": round(gbs, 1), "frac_of_hbm_peak": round(gbs / peaks["hbm_gbs"], 4),
             "shape": dict(rows=rows, hidden=hidden, splits=splits)}
 
@@ -441,9 +450,10 @@ def delta_rule(tokens=2048, batch=1, heads=16, dk=64, dv=128, taps=4, prep=0, he
     return _result("delta_rule (decay per head)" if head else "delta_rule", us, peaks, shape, nbytes, 6.0 * n * heads * dk * dv)
 
 
-def routed_experts(tokens=2048, width=2048, ff=1024, experts=16, top=4, groups=4, keep=3, mma=1, iters=5, peaks=None):
+def routed_experts(tokens=2048, width=2048, ff=1024, experts=16, top=4, groups=4, keep=3, mma=1, clamped=0, iters=5,
+                   peaks=None):
     """Routing, sorting the pairs by expert, both expert products and the weighted sum of ``tokens`` tokens
-    (``mma=0``: the CUDA-core products)."""
+    (``mma=0``: the CUDA-core products; ``clamped``: a clamped gate and the weights on the experts' inputs)."""
     from gllm_b200 import ops
     from gllm_b200.ops import moe
 
@@ -460,7 +470,8 @@ def routed_experts(tokens=2048, width=2048, ff=1024, experts=16, top=4, groups=4
 
     def fn():
         ids, weights = moe.route(logits, correction, top, groups, keep)
-        return moe.apply_experts(x, ids, weights, w_gu, w_d, None, tensor_cores)
+        return moe.apply_experts(x, ids, weights, w_gu, w_d, None, tensor_cores,
+                                 act=(1.702, 7.0, 1.0) if clamped else moe.PLAIN_GATE, weight_on_input=bool(clamped))
 
     us = _time(fn, iters, flush)
     used = min(experts, tokens * top)
@@ -615,6 +626,31 @@ def rope_store(tokens=2048, batch=1, context=0, hq=32, hkv=8, d=64, block_size=1
                    n * 2 * (hq + 2 * hkv) * d * 2)
 
 
+def conv_qkv(tokens=2048, batch=1, context=0, hq=32, hkv=8, d=64, taps=4, splits=0, own=1, block_size=16, iters=5,
+             peaks=None):
+    """Bias, convolution over time, head norms, rotation and store: the kernel between the fused projection (a tensor, or
+    ``splits`` unsummed fp32 parts) and the attention (``own=0``: queries alone)."""
+    from gllm_b200 import ops
+    from gllm_b200.ops.conv_qkv import conv_qkv as kernel
+
+    b = _Batch(batch, tokens, context)
+    pool, table = _paged_cache(batch, context + tokens, hkv, d, block_size)
+    n, cols = batch * tokens, (hq + (2 * hkv if own else 0)) * d
+    parts = torch.randn(max(splits, 1), n, cols, device="cuda")
+    proj = ops.SplitSum(parts, torch.bfloat16) if splits else parts[0].to(torch.bfloat16)
+    page = table[b.token_row.long(), (b.positions // block_size).long()]
+    slots = (page * block_size + b.positions % block_size).to(torch.int32)
+    ones, freq = torch.ones(d, device="cuda"), torch.rand(d // 2, device="cuda")
+    conv_w, bias = torch.randn(taps, cols, device="cuda"), torch.zeros(cols, device="cuda")
+    state = torch.zeros(batch + 1, taps - 1, cols, device="cuda")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    us = _time(lambda: kernel(proj, bias, conv_w, state, ones, ones, 1e-5, freq, d, 1.1, slots, pool, hq, hkv, d, d, d, b,
+                              own_kv=bool(own)), iters, flush)
+    return _result("conv_qkv", us, peaks, dict(tokens=tokens, batch=batch, heads=hq, kv_heads=hkv, head_dim=d, taps=taps,
+                                               splits=splits, own=own),
+                   n * cols * ((4 * splits if splits else 2) + 2) + batch * 2 * (taps - 1) * cols * 4 + cols * 4 * (taps + 1))
+
+
 def depth_conv(tokens=2048, batch=1, hidden=2048, taps=4, streams=0, splits=0, iters=5, peaks=None):
     """The kernel between two sublayers: norm and add of the sublayer's result (a tensor, or ``splits`` unsummed fp32
     parts), the average over ``streams`` earlier streams (0: none), the convolution over time."""
@@ -643,6 +679,7 @@ def depth_conv(tokens=2048, batch=1, hidden=2048, taps=4, streams=0, splits=0, i
 KERNELS = {
     "distance_attention": distance_attention,
     "depth_conv": depth_conv,
+    "conv_qkv": conv_qkv,
     "rope_store": rope_store,
     "differential_attention": differential_attention,
     "step_sized_recurrence": step_sized_recurrence,

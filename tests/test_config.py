@@ -133,3 +133,5 @@ def test_presets_parse():
     assert wide.architecture == "Sazisun" and wide.hidden_size == 2048 and wide.layers[3].mixer["kv_from"] == 1
     wide = load_config(load_preset("vonedra-w2048"))
     assert wide.architecture == "Vonedra" and wide.conv_taps == 4 and wide.value_mixing_layers() == [0, 3]
+    wide = load_config(load_preset("pifelix-w2048"))
+    assert wide.architecture == "Pifelix" and wide.hidden_size == 2048 and wide.layers[5].mixer["kv_from"] == 3
