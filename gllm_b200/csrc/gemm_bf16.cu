@@ -266,6 +266,8 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
       const int kb_end = min(num_kb_total, kb_begin + kb_per_split);
       const bool has_k = kb_end > kb_begin;
       const uint32_t acc = n_used & 1u;
+      float rs = 1.f;                                    // (requested before the wait)
+      if (GATED && !SWAPPED && groups.row_scale != nullptr && item.a_row0 + row < M) rs = groups.row_scale[item.a_row0 + row];
       if (has_k) {
         mbar_wait(smem_addr(&tmem_full_bar[acc]), (n_used >> 1) & 1u, status, &abort_flag);
         // the four warps leave together: one that gave up has set abort_flag before this barrier
@@ -280,7 +282,6 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
         if (!SWAPPED) {
           // this thread's token row holds, per 128 columns, 64 gates then their 64 ups
           const int m = item.a_row0 + row;
-          const float rs = groups.row_scale != nullptr && m < M ? groups.row_scale[m] : 1.f;
 #pragma unroll 1
           for (int c2 = 0; c2 < BN / 2; c2 += 16) {
             const int gate_col = (c2 / 64) * 128 + (c2 % 64);
