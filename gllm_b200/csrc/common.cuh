@@ -40,6 +40,14 @@ __device__ __forceinline__ float gate_act(float g, float u, const GateAct& a) {
   }
   return g / (1.0f + __expf(-a.slope * g)) * (u + a.offset);
 }
+// The same for results that are rounded to bfloat16 at once: the division within 2 ulp (0 for a huge divisor).
+__device__ __forceinline__ float gate_act_bf16(float g, float u, const GateAct& a) {
+  if (a.limit > 0.f) {
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+  }
+  return __fdividef(g, 1.0f + __expf(-a.slope * g)) * (u + a.offset);
+}
 
 // The first key position a query at position p sees, whatever kind of bound the layer has: `window` > 0 keeps the last
 // `window` positions, `window` < 0 cuts the sequence into chunks of -window positions counted from position 0 and keeps

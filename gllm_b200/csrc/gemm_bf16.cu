@@ -292,7 +292,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             if (m < M && f0 < n_out) {
               float y[16];
 #pragma unroll
-              for (int i = 0; i < 16; ++i) y[i] = gate_act(g[i] * rs, u[i] * rs, act);
+              for (int i = 0; i < 16; ++i) y[i] = gate_act_bf16(g[i] * rs, u[i] * rs, act);
               OutT* dst = out + (int64_t)m * ldo + f0;
               if (f0 + 16 <= n_out && sizeof(OutT) == 2 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
                 uint4 p0, p1;
@@ -338,7 +338,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 if (m < M) {
                   const float mine_v = row < 64 ? v[i] : v[CH - 16 + i], other = exch[row & 63][c + off + i];
                   const float g = row < 64 ? mine_v : other, u = row < 64 ? other : mine_v;
-                  out[(int64_t)m * ldo + f] = cast_out<OutT>(gate_act(g, u, act));
+                  out[(int64_t)m * ldo + f] = cast_out<OutT>(gate_act_bf16(g, u, act));
                 }
               }
             }

@@ -236,7 +236,7 @@ umma_gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_co
           if (m < M && f0 < n_out) {
             float y[16];
 #pragma unroll
-            for (int i = 0; i < 16; ++i) y[i] = gate_act(g[i], u[i], act);
+            for (int i = 0; i < 16; ++i) y[i] = gate_act_bf16(g[i], u[i], act);
             OutT* dst = out + (int64_t)m * ldo + f0;
             if (f0 + 16 <= n_out && sizeof(OutT) == 2 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
               uint4 p0, p1;
