@@ -67,7 +67,7 @@ struct Item {
   int w_row0;      // first weight row of the tile in the weight's tensor map (b_row0, or that row of the tile's group)
   bool skip;       // grouped: a tile of rows behind the last one in use
 };
-// Grouped products (normal orientation only): the rows of X come in tiles of BM that each belong to one group
+// Grouped products: the rows of X come in tiles of BM (swapped: BN) that each belong to one group
 // (``group_of_tile[tile]``, ``num_tiles[0]`` tiles in use, both written on the device by the kernel before this one),
 // and group g multiplies by rows g * group_rows .. of W.  N is then the rows of ONE group.
 struct Groups {
@@ -94,10 +94,10 @@ __device__ __forceinline__ Item item_of(int w, int tiles_a, int splits) {
 template <int BN, bool SWAPPED>
 __device__ __forceinline__ Item item_of(int w, int tiles_a, int splits, const Groups& groups) {
   Item it = item_of<BN, SWAPPED>(w, tiles_a, splits);
-  if (!SWAPPED && groups.group_of_tile != nullptr) {
-    const int ta = it.a_row0 / BM;
-    it.skip = ta >= groups.num_tiles[0];
-    if (!it.skip) it.w_row0 += groups.group_of_tile[ta] * groups.group_rows;
+  if (groups.group_of_tile != nullptr) {
+    const int tile = SWAPPED ? it.b_row0 / BN : it.a_row0 / BM;
+    it.skip = tile >= groups.num_tiles[0];
+    if (!it.skip) it.w_row0 += groups.group_of_tile[tile] * groups.group_rows;
   }
   return it;
 }
@@ -337,7 +337,8 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 const int m = item.b_row0 + c + off + i;
                 if (m < M) {
                   const float mine_v = row < 64 ? v[i] : v[CH - 16 + i], other = exch[row & 63][c + off + i];
-                  const float g = row < 64 ? mine_v : other, u = row < 64 ? other : mine_v;
+                  const float rw = groups.row_scale != nullptr ? groups.row_scale[m] : 1.f;
+                  const float g = (row < 64 ? mine_v : other) * rw, u = (row < 64 ? other : mine_v) * rw;
                   out[(int64_t)m * ldo + f] = cast_out<OutT>(gate_act_bf16(g, u, act));
                 }
               }
@@ -637,18 +638,22 @@ GLLM_API int gllm_gemm_bf16_accumulate(const __nv_bfloat16* X, const __nv_bfloat
 #undef GLLM_ACC
 }
 
-// Grouped product: the rows of X [rows, K] come in tiles of 128 that each belong to one group (``group_of_tile``,
-// ``num_tiles`` on the device); group g multiplies by W[g] of W [groups, N, K].  gated != 0: W[g]'s rows are blocks of
-// 64 gate rows and the 64 up rows of the same features and out is bf16 [rows, N / 2], the gated activation of the two
-// (slope, limit, offset as gllm_gemm_bf16_gated takes them; row_scale, null or [rows]: gate and up are multiplied by the
-// row's number first); otherwise out is fp32 [rows, N].  Rows of tiles behind ``num_tiles[0]`` are neither read nor written; a row of X that no pair
-// owns gives a row of out that nobody reads (rows do not mix).
+// Grouped product: the rows of X [rows, K] come in tiles of `tile_rows` (128, or 16, 32, 64 for few rows per group: the
+// weight is then the 128-row operand) that each belong to one group (``group_of_tile``, ``num_tiles`` on the device);
+// group g multiplies by W[g] of W [groups, N, K].  gated != 0: W[g]'s rows are blocks of 64 gate rows and the 64 up rows
+// of the same features and out is bf16 [rows, N / 2], the gated activation of the two (slope, limit, offset as
+// gllm_gemm_bf16_gated takes them; row_scale, null or [rows]: gate and up are multiplied by the row's number first);
+// otherwise out is fp32 [rows, N], or with splits > 1 (small tiles only) [splits][rows, N], every range of K by itself.
+// Rows of tiles behind ``num_tiles[0]`` are neither read nor written; a row of X that no pair owns gives a row of out
+// that nobody reads (rows do not mix).
 GLLM_API int gllm_gemm_bf16_grouped(const __nv_bfloat16* X, const __nv_bfloat16* W, void* out, int gated, int rows, int N,
                                     int K, int groups, const int* group_of_tile, const int* num_tiles, int wide,
-                                    const float* row_scale, float slope, float limit, float offset, int* status,
-                                    cudaStream_t stream) {
+                                    const float* row_scale, float slope, float limit, float offset, int tile_rows,
+                                    int splits, int* status, cudaStream_t stream) {
   if (rows <= 0 || N <= 0 || groups <= 0) return 0;
-  if (rows % BM || K <= 0 || K % 8 || (gated && N % 128) || (reinterpret_cast<uintptr_t>(X) & 15) ||
+  const bool few = tile_rows == 16 || tile_rows == 32 || tile_rows == 64;
+  if ((!few && tile_rows != BM) || splits < 1 || splits > 16 || (splits > 1 && (gated || !few))) return (int)cudaErrorInvalidValue;
+  if (rows % tile_rows || K <= 0 || K % 8 || (gated && N % 128) || (reinterpret_cast<uintptr_t>(X) & 15) ||
       (reinterpret_cast<uintptr_t>(W) & 15) || (int64_t)groups * N > 0x7fffffff)
     return (int)cudaErrorInvalidValue;
   if (row_scale != nullptr && !gated) return (int)cudaErrorInvalidValue;
@@ -658,6 +663,18 @@ GLLM_API int gllm_gemm_bf16_grouped(const __nv_bfloat16* X, const __nv_bfloat16*
 #define GLLM_GROUPED(BN, OutT, GATED, ldo) \
   return umma_launch<BN, false, OutT, GATED>(X, W, (OutT*)out, rows, N, K, K, K, ldo, 1, nullptr, nullptr, 0, status, \
                                              stream, 0, act, g, w_rows)
+#define GLLM_GROUPED_FEW(BN)                                                                                            \
+  {                                                                                                                    \
+    if (gated)                                                                                                         \
+      return umma_launch<BN, true, __nv_bfloat16, true>(X, W, (__nv_bfloat16*)out, rows, N, K, K, K, N / 2, 1, nullptr,  \
+                                                        nullptr, 0, status, stream, 0, act, g, w_rows);                \
+    return umma_launch<BN, true, float, false>(X, W, (float*)out, rows, N, K, K, K, N, splits, (float*)out, nullptr, 0, \
+                                               status, stream, 0, act, g, w_rows);                                     \
+  }
+  if (tile_rows == 16) GLLM_GROUPED_FEW(16);
+  if (tile_rows == 32) GLLM_GROUPED_FEW(32);
+  if (tile_rows == 64) GLLM_GROUPED_FEW(64);
+#undef GLLM_GROUPED_FEW
   if (gated) {
     if (wide && N % 256 == 0) GLLM_GROUPED(256, __nv_bfloat16, true, N / 2);
     GLLM_GROUPED(128, __nv_bfloat16, true, N / 2);

@@ -6,9 +6,11 @@
 //                `group_max`; experts of other groups
 //                count as minus infinity); the weights are the chosen experts' s (divided by their sum + renorm_eps with
 //                `renorm`), times `weight_scale`.  Ties go to the lower index.
+//                (the logits may come as unsummed splits of their product)
 //   moe_align    (one block) sorts the (token, slot) pairs by expert: every expert's pairs form whole tiles of
 //                `tile_m` rows (the last one filled up with -1), so that a tile of the products below reads ONE
 //                expert's weights; writes the pair of every row, the expert of every tile and the tile count.
+//   moe_route_align  both in one launch of one block, for few tokens.
 //   moe_gemm     out[pair] = A[row of pair] @ W[expert]^T over the tiles; `gated`: W holds gate and up rows and
 //                the result is the gated activation of the two (GateAct: silu(gate) * up, or with a slope, clamps and
 //                an offset), rounded to T; `act` 1 (experts without a gate): the square of
@@ -21,7 +23,10 @@
 // A pair's result does not depend on which other pairs share its tile or on the tile's place: every row is a dot
 // product over K in one fixed order.  Scores, choice, weights, accumulators and the combination are fp32.
 #include "common.cuh"
+#include "row_sum.cuh"
 #include <math_constants.h>
+
+#include <algorithm>
 
 namespace {
 
@@ -37,36 +42,48 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
-__global__ void __launch_bounds__(32)
-moe_route_kernel(const float* __restrict__ logits, int64_t stride, const float* __restrict__ correction,
-                 int* __restrict__ ids, float* __restrict__ weights, int experts, int top, int groups, int keep,
-                 int renorm, int softmax_scores, int group_max, float renorm_eps, float weight_scale) {
-  extern __shared__ float sm[];
+// Router logits of one product: [n, experts] at `stride`, or up to 16 unsummed splits of it, summed in ascending order.
+struct RouterLogits {
+  const float* z;
+  int64_t stride;
+  int n_parts;              // 0: not split
+  int64_t part_stride;
+  __device__ __forceinline__ float at(int64_t i, int e) const {
+    const float* p = z + i * stride + e;
+    return n_parts ? sum_parts16(p, n_parts, part_stride) : *p;
+  }
+};
+struct RouteRule {
+  int experts, top, groups, keep, renorm, softmax_scores, group_max;
+  float renorm_eps, weight_scale;
+};
+
+// Token i by one warp; sm: 2 * experts + groups floats of shared memory of this warp's own.
+__device__ __forceinline__ void route_token(const RouterLogits& logits, const float* __restrict__ correction,
+                                            int* ids, float* weights, int i, const RouteRule& rule, float* sm) {
+  const int experts = rule.experts, groups = rule.groups, lane = threadIdx.x & 31;
   float* s = sm;                 // [experts] scores
   float* c = s + experts;        // [experts] choice scores
   float* gs = c + experts;       // [groups] group scores, then 1 = kept
-  pdl_trigger();
-  pdl_wait();
-  const int i = blockIdx.x, lane = threadIdx.x;
+  for (int e = lane; e < experts; e += 32) s[e] = logits.at(i, e);
   float z_max = -CUDART_INF_F, z_sum = 0.f;
-  if (softmax_scores) {
-    for (int e = lane; e < experts; e += 32) z_max = fmaxf(z_max, logits[(int64_t)i * stride + e]);
+  if (rule.softmax_scores) {
+    for (int e = lane; e < experts; e += 32) z_max = fmaxf(z_max, s[e]);
     z_max = warp_max(z_max);
     for (int e = lane; e < experts; e += 32) {
-      const float v = expf(logits[(int64_t)i * stride + e] - z_max);
+      const float v = expf(s[e] - z_max);
       s[e] = v;
       z_sum += v;
     }
     z_sum = warp_sum(z_sum);
   }
   for (int e = lane; e < experts; e += 32) {
-    const float z = logits[(int64_t)i * stride + e];
-    const float v = softmax_scores ? s[e] / z_sum : 1.0f / (1.0f + expf(-z));
+    const float v = rule.softmax_scores ? s[e] / z_sum : 1.0f / (1.0f + expf(-s[e]));
     s[e] = v;
     c[e] = v + (correction ? correction[e] : 0.f);
   }
   __syncwarp();
-  if (groups > 1 && keep < groups) {
+  if (groups > 1 && rule.keep < groups) {
     const int per = experts / groups;
     for (int g = lane; g < groups; g += 32) {
       float m1 = -CUDART_INF_F, m2 = -CUDART_INF_F;
@@ -79,11 +96,11 @@ moe_route_kernel(const float* __restrict__ logits, int64_t stride, const float* 
           m2 = v;
         }
       }
-      gs[g] = (per > 1 && !group_max) ? m1 + m2 : m1;
+      gs[g] = (per > 1 && !rule.group_max) ? m1 + m2 : m1;
     }
     __syncwarp();
     // the `keep` best groups, one after the other; a kept group is marked by +inf ... then turned into a flag
-    for (int r = 0; r < keep; ++r) {
+    for (int r = 0; r < rule.keep; ++r) {
       float best = -CUDART_INF_F;
       int bi = 0x7fffffff;
       for (int g = lane; g < groups; g += 32) {
@@ -103,7 +120,7 @@ moe_route_kernel(const float* __restrict__ logits, int64_t stride, const float* 
     __syncwarp();
   }
   float total = 0.f;
-  for (int r = 0; r < top; ++r) {
+  for (int r = 0; r < rule.top; ++r) {
     float best = -CUDART_INF_F;
     int bi = 0x7fffffff;
     for (int e = lane; e < experts; e += 32) {
@@ -117,33 +134,38 @@ moe_route_kernel(const float* __restrict__ logits, int64_t stride, const float* 
     __syncwarp();
     if (bi >= experts) bi = 0;              // nothing left to choose (NaN logits): keep the indices in range
     if (lane == 0) {
-      ids[(int64_t)i * top + r] = bi;
-      weights[(int64_t)i * top + r] = s[bi];
+      ids[(int64_t)i * rule.top + r] = bi;
+      weights[(int64_t)i * rule.top + r] = s[bi];
       c[bi] = -CUDART_INF_F;
     }
     total += s[bi];
     __syncwarp();
   }
-  if (renorm || weight_scale != 1.0f) {
+  if (rule.renorm || rule.weight_scale != 1.0f) {
     __syncwarp();
-    for (int r = lane; r < top; r += 32) {
-      float wv = weights[(int64_t)i * top + r];
-      if (renorm) wv /= total + renorm_eps;
-      weights[(int64_t)i * top + r] = wv * weight_scale;
+    for (int r = lane; r < rule.top; r += 32) {
+      float wv = weights[(int64_t)i * rule.top + r];
+      if (rule.renorm) wv /= total + rule.renorm_eps;
+      weights[(int64_t)i * rule.top + r] = wv * rule.weight_scale;
     }
   }
+  __syncwarp();
 }
 
-__global__ void __launch_bounds__(1024)
-moe_align_kernel(const int* __restrict__ ids, int* __restrict__ sorted, int* __restrict__ tile_expert,
-                 int* __restrict__ num_tiles, int* __restrict__ row_of_pair, int n_pairs, int experts, int tile_m,
-                 int max_tiles) {
-  extern __shared__ int smi[];
+__global__ void __launch_bounds__(32)
+moe_route_kernel(RouterLogits logits, const float* __restrict__ correction, int* ids, float* weights, RouteRule rule) {
+  extern __shared__ float sm[];
+  pdl_trigger();
+  pdl_wait();
+  route_token(logits, correction, ids, weights, blockIdx.x, rule, sm);
+}
+
+// By one block; smi: 3 * experts + 1 ints of shared memory.
+__device__ __forceinline__ void align_pairs(const int* ids, int* sorted, int* tile_expert, int* num_tiles, int* row_of_pair,
+                                            int n_pairs, int experts, int tile_m, int max_tiles, int* smi) {
   int* counts = smi;                  // [experts]
   int* first = counts + experts;      // [experts + 1] first row of every expert
   int* cursor = first + experts + 1;  // [experts]
-  pdl_trigger();
-  pdl_wait();
   for (int e = threadIdx.x; e < experts; e += blockDim.x) counts[e] = cursor[e] = 0;
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
@@ -163,15 +185,41 @@ moe_align_kernel(const int* __restrict__ ids, int* __restrict__ sorted, int* __r
   __syncthreads();
   for (int e = threadIdx.x; e < experts; e += blockDim.x)
     for (int t = first[e] / tile_m; t < first[e + 1] / tile_m && t < max_tiles; ++t) tile_expert[t] = e;
-  for (int r = threadIdx.x; r < max_tiles * tile_m; r += blockDim.x) sorted[r] = -1;
+  if (sorted)
+    for (int r = threadIdx.x; r < max_tiles * tile_m; r += blockDim.x) sorted[r] = -1;
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
     const int e = ids[p];
     if (e < 0 || e >= experts) continue;
     const int row = first[e] + atomicAdd(&cursor[e], 1);
-    if (row < max_tiles * tile_m) sorted[row] = p;
+    if (sorted && row < max_tiles * tile_m) sorted[row] = p;
     if (row_of_pair) row_of_pair[p] = min(row, max_tiles * tile_m - 1);
   }
+}
+
+__global__ void __launch_bounds__(1024)
+moe_align_kernel(const int* __restrict__ ids, int* __restrict__ sorted, int* __restrict__ tile_expert,
+                 int* __restrict__ num_tiles, int* __restrict__ row_of_pair, int n_pairs, int experts, int tile_m,
+                 int max_tiles) {
+  extern __shared__ int smi[];
+  pdl_trigger();
+  pdl_wait();
+  align_pairs(ids, sorted, tile_expert, num_tiles, row_of_pair, n_pairs, experts, tile_m, max_tiles, smi);
+}
+
+// Both for few tokens, by one block: a warp per token in turn, then the sort.
+__global__ void __launch_bounds__(1024)
+moe_route_align_kernel(RouterLogits logits, const float* __restrict__ correction, int* ids, float* weights, RouteRule rule,
+                       int n_tokens, int* sorted, int* tile_expert, int* num_tiles, int* row_of_pair, int tile_m,
+                       int max_tiles) {
+  extern __shared__ float sm[];
+  pdl_trigger();
+  pdl_wait();
+  const int per_warp = 2 * rule.experts + rule.groups, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  for (int i = warp; i < n_tokens; i += nwarps) route_token(logits, correction, ids, weights, i, rule, sm + warp * per_warp);
+  __syncthreads();
+  align_pairs(ids, sorted, tile_expert, num_tiles, row_of_pair, n_tokens * rule.top, rule.experts, tile_m, max_tiles,
+              reinterpret_cast<int*>(sm + nwarps * per_warp));
 }
 
 // out[row_of_pair[p]] = x[p / top]: the tokens' rows in the order of the sorted pairs (and, with row_scale, the pairs'
@@ -273,23 +321,23 @@ moe_gemm_kernel(const T* __restrict__ a, int64_t a_stride, int a_div, const T* _
   }
 }
 
-template <typename T>
+// A thread takes VEC neighbouring columns; the rows of up to four slots are requested together.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ weights, const T* __restrict__ shared,
-                   T* __restrict__ out, const int* __restrict__ row_of_pair, int top, int width,
+moe_combine_kernel(RowSum y, const T* __restrict__ shared, T* __restrict__ out, int width,
                    const float* __restrict__ shared_gate, int64_t shared_gate_stride) {
   pdl_trigger();
   pdl_wait();
   const int64_t t = blockIdx.x;
   const float sg = (shared && shared_gate) ? 1.0f / (1.0f + expf(-shared_gate[t * shared_gate_stride])) : 1.0f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    float acc = 0.f;
-    for (int s = 0; s < top; ++s) {
-      const int64_t row = row_of_pair ? (int64_t)row_of_pair[t * top + s] : t * top + s;
-      acc = fmaf(weights ? weights[t * top + s] : 1.f, y[row * width + c], acc);
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; c < width; c += gridDim.y * blockDim.x * VEC) {
+    float acc[VEC];
+    y.sum<VEC>(t, c, width, acc);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      if (shared) acc[e] = fmaf(sg, to_float(shared[t * width + c + e]), acc[e]);
+      out[t * width + c + e] = from_float<T>(acc[e]);
     }
-    if (shared) acc = fmaf(sg, to_float(shared[t * width + c]), acc);
-    out[t * width + c] = from_float<T>(acc);
   }
 }
 
@@ -319,17 +367,22 @@ int moe_gemm_launch(const T* a, int64_t a_stride, int a_div, const T* w, int64_t
 }
 }  // namespace
 
-GLLM_API int gllm_moe_route(const float* logits, int64_t stride, const float* correction, int* ids, float* weights,
-                            int n_tokens, int experts, int top, int groups, int keep, int renorm, int softmax_scores,
-                            int group_max, float renorm_eps, float weight_scale, cudaStream_t stream) {
+static bool rule_ok(const RouteRule& r) {
+  return r.experts >= 1 && r.top >= 1 && r.top <= r.experts && r.groups >= 1 && r.experts % r.groups == 0 && r.keep >= 1 &&
+         r.keep <= r.groups && r.top <= r.keep * (r.experts / r.groups);
+}
+
+// logits: [n, experts] at `stride`; n_parts > 0: that many unsummed fp32 splits of it, part_stride floats apart.
+GLLM_API int gllm_moe_route(const float* logits, int64_t stride, int n_parts, int64_t part_stride, const float* correction,
+                            int* ids, float* weights, int n_tokens, int experts, int top, int groups, int keep, int renorm,
+                            int softmax_scores, int group_max, float renorm_eps, float weight_scale,
+                            cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (experts < 1 || top < 1 || top > experts || groups < 1 || experts % groups || keep < 1 || keep > groups ||
-      top > keep * (experts / groups))
-    return (int)cudaErrorInvalidValue;
+  const RouteRule rule{experts, top, groups, keep, renorm, softmax_scores, group_max, renorm_eps, weight_scale};
   const size_t smem = sizeof(float) * (size_t)(2 * experts + groups);
-  if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-  return gllm_launch(moe_route_kernel, dim3(n_tokens), dim3(32), smem, stream, logits, stride, correction, ids, weights,
-                     experts, top, groups, keep, renorm, softmax_scores, group_max, renorm_eps, weight_scale);
+  if (!rule_ok(rule) || n_parts > 16 || smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+  return gllm_launch(moe_route_kernel, dim3(n_tokens), dim3(32), smem, stream,
+                     RouterLogits{logits, stride, n_parts, part_stride}, correction, ids, weights, rule);
 }
 
 GLLM_API int gllm_moe_align(const int* ids, int* sorted, int* tile_expert, int* num_tiles, int* row_of_pair,
@@ -339,6 +392,22 @@ GLLM_API int gllm_moe_align(const int* ids, int* sorted, int* tile_expert, int* 
   if (smem > 48 * 1024 || tile_m < 1 || max_tiles < 1) return (int)cudaErrorInvalidValue;
   return gllm_launch(moe_align_kernel, dim3(1), dim3(1024), smem, stream, ids, sorted, tile_expert, num_tiles, row_of_pair,
                      n_pairs, experts, tile_m, max_tiles);
+}
+
+// Routing and sorting in one launch of one block, for few tokens (the experts' scores of all warps fit 48 KB).
+GLLM_API int gllm_moe_route_align(const float* logits, int64_t stride, int n_parts, int64_t part_stride,
+                                  const float* correction, int* ids, float* weights, int n_tokens, int experts, int top,
+                                  int groups, int keep, int renorm, int softmax_scores, int group_max, float renorm_eps,
+                                  float weight_scale, int* sorted, int* tile_expert, int* num_tiles, int* row_of_pair,
+                                  int tile_m, int max_tiles, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  const RouteRule rule{experts, top, groups, keep, renorm, softmax_scores, group_max, renorm_eps, weight_scale};
+  const int warps = std::min(32, std::max(4, n_tokens));
+  const size_t smem = sizeof(float) * (size_t)warps * (2 * experts + groups) + sizeof(int) * (size_t)(3 * experts + 1);
+  if (!rule_ok(rule) || n_parts > 16 || smem > 48 * 1024 || tile_m < 1 || max_tiles < 1) return (int)cudaErrorInvalidValue;
+  return gllm_launch(moe_route_align_kernel, dim3(1), dim3(warps * 32), smem, stream,
+                     RouterLogits{logits, stride, n_parts, part_stride}, correction, ids, weights, rule, n_tokens, sorted,
+                     tile_expert, num_tiles, row_of_pair, tile_m, max_tiles);
 }
 
 GLLM_API int gllm_moe_gemm_f32(const float* a, int64_t a_stride, int a_div, const float* w, int64_t w_expert_stride,
@@ -358,20 +427,30 @@ GLLM_API int gllm_moe_gemm_bf16(const __nv_bfloat16* a, int64_t a_stride, int a_
                                         GateAct{slope, limit, offset}, stream);
 }
 
-GLLM_API int gllm_moe_combine_f32(const float* y, const float* weights, const float* shared, float* out,
-                                  const int* row_of_pair, int n_tokens, int top, int width, const float* shared_gate,
-                                  int64_t shared_gate_stride, cudaStream_t stream) {
+template <typename T>
+static int moe_combine_launch(const float* y, int n_parts, int64_t part_stride, const float* weights, const T* shared, T* out,
+                              const int* row_of_pair, int n_tokens, int top, int width, const float* shared_gate,
+                              int64_t shared_gate_stride, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  return gllm_launch(moe_combine_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, y, weights, shared, out,
-                     row_of_pair, top, width, shared_gate, shared_gate_stride);
+  if (n_parts < 1 || top < 1 || width < 1) return (int)cudaErrorInvalidValue;
+  const RowSum rows{y, n_parts, part_stride, row_of_pair, weights, top};
+  const bool vec = width % 4 == 0 && part_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+  const int blocks_y = n_tokens >= 64 ? 1 : (width + (vec ? 1024 : 256) - 1) / (vec ? 1024 : 256);
+  auto kernel = vec ? moe_combine_kernel<T, 4> : moe_combine_kernel<T, 1>;
+  return gllm_launch(kernel, dim3(n_tokens, blocks_y), dim3(256), 0, stream, rows, shared, out, width, shared_gate,
+                     shared_gate_stride);
 }
-GLLM_API int gllm_moe_combine_bf16(const float* y, const float* weights, const __nv_bfloat16* shared,
-                                   __nv_bfloat16* out, const int* row_of_pair, int n_tokens, int top, int width,
-                                   const float* shared_gate, int64_t shared_gate_stride, cudaStream_t stream) {
-  if (n_tokens <= 0) return 0;
-  return gllm_launch(moe_combine_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, stream, y, weights, shared, out,
-                     row_of_pair, top, width, shared_gate, shared_gate_stride);
-}
+// y: [n_parts][rows, width] fp32, the parts added in ascending order first.
+#define GLLM_MOE_COMBINE(T, S)                                                                                         \
+  GLLM_API int gllm_moe_combine_##S(const float* y, int n_parts, int64_t part_stride, const float* weights,            \
+                                    const T* shared, T* out, const int* row_of_pair, int n_tokens, int top, int width, \
+                                    const float* shared_gate, int64_t shared_gate_stride, cudaStream_t stream) {       \
+    return moe_combine_launch<T>(y, n_parts, part_stride, weights, shared, out, row_of_pair, n_tokens, top, width,     \
+                                 shared_gate, shared_gate_stride, stream);                                             \
+  }
+GLLM_MOE_COMBINE(float, f32)
+GLLM_MOE_COMBINE(__nv_bfloat16, bf16)
+
 GLLM_API int gllm_moe_gather_bf16(const __nv_bfloat16* x, int64_t x_stride, const int* row_of_pair, __nv_bfloat16* out,
                                   int n_pairs, int top, int width, const float* weights, float* row_scale,
                                   cudaStream_t stream) {

@@ -2,13 +2,15 @@
 //   resid[r] += value[r] / sqrt(mean(value[r]^2) + post_eps) * post_w  (+ extra[r]);   out[r] = rms(resid[r]) * w
 // (without post_w the value is added as it is; value and extra may each be absent) in one pass over the row: the add that the pre-norm layers defer to the next norm's kernel is deferred here
 // as well, together with the norm of what is added.  `value` may arrive as unsummed fp32 splits of a product
-// (summed in ascending order and rounded to T, as the product would have); `extra` is a second fp32 stream
+// (summed in ascending order and rounded to T, as the product would have), or as the rows of routed experts that are
+// still to be added up per token (RowSum, rounded to T); `extra` is a second fp32 stream
 // that is added as it is (the embedding output that a repeated stretch of layers takes in again).  With
 // `rows` only those rows are normed and resid stays untouched (the final norm at the wanted rows).
 // Without w nothing is normed on the way out: out[r] is the new resid[r] rounded to T (layers whose sublayers read the
 // residual itself).
 // Statistics, the normed value and the sums are fp32 whatever T is.
 #include "common.cuh"
+#include "row_sum.cuh"
 
 namespace {
 
@@ -52,21 +54,26 @@ __global__ void __launch_bounds__(1024)
 postnorm_add_rmsnorm_kernel(const T* __restrict__ value, const float* __restrict__ parts, int n_parts,
                             int64_t part_stride, const float* __restrict__ post_w, float post_eps,
                             const float* __restrict__ extra, float* __restrict__ resid, const float* __restrict__ w,
-                            float eps, T* __restrict__ out, const int* __restrict__ rows, int n_rows, int hidden) {
+                            float eps, T* __restrict__ out, const int* __restrict__ rows, int n_rows, int hidden,
+                            RowSum row_sum) {
   extern __shared__ __align__(16) float xs[];
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
   const int64_t r = rows ? rows[blockIdx.x] : blockIdx.x;
   float* x = resid + r * hidden;
-  const bool has_value = value != nullptr || parts != nullptr;
+  const bool has_value = value != nullptr || parts != nullptr || row_sum.y != nullptr;
   const int first = threadIdx.x * VEC, stride = blockDim.x * VEC;
   float inv1 = 1.f;
   if (has_value) {
     float ss = 0.f;
     for (int c = first; c < hidden; c += stride) {
       float v[VEC];
-      if (parts) {
+      if (row_sum.y) {
+        row_sum.sum<VEC>(r, c, hidden, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = to_float(from_float<T>(v[e]));
+      } else if (parts) {
 #pragma unroll
         for (int e = 0; e < VEC; ++e)
           v[e] = to_float(from_float<T>(sum_parts16(parts + r * hidden + c + e, n_parts, part_stride)));
@@ -128,14 +135,15 @@ postnorm_add_rmsnorm_kernel(const T* __restrict__ value, const float* __restrict
 template <typename T>
 int postnorm_launch(const T* value, const float* parts, int n_parts, int64_t part_stride, const float* post_w,
                     float post_eps, const float* extra, float* resid, const float* w, float eps, T* out,
-                    const int* rows, int n_rows, int hidden, cudaStream_t stream) {
+                    const int* rows, int n_rows, int hidden, const RowSum& row_sum, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   const size_t smem = sizeof(float) * (size_t)hidden;
   if (smem > 200 * 1024 || n_parts > 16) return (int)cudaErrorInvalidValue;
   auto misaligned = [](const void* p) { return p != nullptr && (reinterpret_cast<uintptr_t>(p) & 15) != 0; };
   const bool vec = hidden % 4 == 0 && !misaligned(value) && !misaligned(post_w) && !misaligned(extra) &&
                    !misaligned(resid) && !misaligned(w) && !misaligned(out) &&
-                   (value == nullptr || (reinterpret_cast<uintptr_t>(value) & 7) == 0);
+                   (value == nullptr || (reinterpret_cast<uintptr_t>(value) & 7) == 0) && !misaligned(row_sum.y) &&
+                   row_sum.part_stride % 4 == 0;
   auto kernel = vec ? postnorm_add_rmsnorm_kernel<T, 4> : postnorm_add_rmsnorm_kernel<T, 1>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -145,22 +153,21 @@ int postnorm_launch(const T* value, const float* parts, int n_parts, int64_t par
   int threads = n_rows <= 64 && hidden > 1024 ? 1024 : 256;
   if (vec) threads = std::max(64, std::min(threads, (hidden / 4 + 31) / 32 * 32));
   return gllm_launch(kernel, dim3(n_rows), dim3(threads), smem, stream, value, parts, n_parts, part_stride, post_w,
-                     post_eps, extra, resid, w, eps, out, rows, n_rows, hidden);
+                     post_eps, extra, resid, w, eps, out, rows, n_rows, hidden, row_sum);
 }
 }  // namespace
 
-GLLM_API int gllm_postnorm_add_rmsnorm_f32(const float* value, const float* parts, int n_parts, int64_t part_stride,
-                                           const float* post_w, float post_eps, const float* extra, float* resid,
-                                           const float* w, float eps, float* out, const int* rows, int n_rows,
-                                           int hidden, cudaStream_t stream) {
-  return postnorm_launch<float>(value, parts, n_parts, part_stride, post_w, post_eps, extra, resid, w, eps, out, rows,
-                                n_rows, hidden, stream);
-}
-GLLM_API int gllm_postnorm_add_rmsnorm_bf16(const __nv_bfloat16* value, const float* parts, int n_parts,
-                                            int64_t part_stride, const float* post_w, float post_eps,
-                                            const float* extra, float* resid, const float* w, float eps,
-                                            __nv_bfloat16* out, const int* rows, int n_rows, int hidden,
-                                            cudaStream_t stream) {
-  return postnorm_launch<__nv_bfloat16>(value, parts, n_parts, part_stride, post_w, post_eps, extra, resid, w, eps, out,
-                                        rows, n_rows, hidden, stream);
-}
+// y, y_parts, y_part_stride, row_of_pair, pair_weights, top: the RowSum (y null: none).
+#define GLLM_POSTNORM(T, S)                                                                                            \
+  GLLM_API int gllm_postnorm_add_rmsnorm_##S(const T* value, const float* parts, int n_parts, int64_t part_stride,     \
+                                             const float* post_w, float post_eps, const float* extra, float* resid,    \
+                                             const float* w, float eps, T* out, const int* rows, int n_rows,           \
+                                             int hidden, const float* y, int y_parts, int64_t y_part_stride,           \
+                                             const int* row_of_pair, const float* pair_weights, int top,               \
+                                             cudaStream_t stream) {                                                    \
+    return postnorm_launch<T>(value, parts, n_parts, part_stride, post_w, post_eps, extra, resid, w, eps, out, rows,   \
+                              n_rows, hidden, RowSum{y, y_parts, y_part_stride, row_of_pair, pair_weights, top},       \
+                              stream);                                                                                 \
+  }
+GLLM_POSTNORM(float, f32)
+GLLM_POSTNORM(__nv_bfloat16, bf16)

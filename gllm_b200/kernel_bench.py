@@ -469,9 +469,9 @@ def routed_experts(tokens=2048, width=2048, ff=1024, experts=16, top=4, groups=4
         w_gu = torch.stack([ops.interleave_gate_up(w[:ff], w[ff:]) for w in w_gu]).contiguous()
 
     def fn():
-        ids, weights = moe.route(logits, correction, top, groups, keep)
-        return moe.apply_experts(x, ids, weights, w_gu, w_d, None, tensor_cores,
-                                 act=(1.702, 7.0, 1.0) if clamped else moe.PLAIN_GATE, weight_on_input=bool(clamped))
+        choice = moe.choose(logits, correction, top, tensor_cores, groups=groups, groups_kept=keep)
+        return moe.apply_choice(x, choice, w_gu, w_d, None, tensor_cores,
+                                act=(1.702, 7.0, 1.0) if clamped else moe.PLAIN_GATE, weight_on_input=bool(clamped))
 
     us = _time(fn, iters, flush)
     used = min(experts, tokens * top)

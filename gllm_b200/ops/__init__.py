@@ -53,6 +53,7 @@ __all__ = [
     "add_dyt",
     "Biased",
     "DepthPending",
+    "RowSum",
 ]
 
 P = c_void_p
@@ -134,7 +135,8 @@ _SIGNATURES = {
                                 c_int, P],
     },
     "postnorm": {
-        "gllm_postnorm_add_rmsnorm_{t}": [P, P, c_int, c_int64, P, c_float, P, P, P, c_float, P, P, c_int, c_int, P],
+        "gllm_postnorm_add_rmsnorm_{t}": [P, P, c_int, c_int64, P, c_float, P, P, P, c_float, P, P, c_int, c_int, P, c_int,
+                                          c_int64, P, P, c_int, P],
     },
     "conv_qkv": {
         "gllm_conv_qkv_{t}": [P, c_int64, P, c_int, c_int64, P, P, P, P, P, P, P, P, c_float, P, c_int, c_float, P, P,
@@ -150,12 +152,14 @@ _SIGNATURES = {
         "gllm_delta_rule": [P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P],
     },
     "moe": {
-        "gllm_moe_route": [P, c_int64, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                           P],
+        "gllm_moe_route": [P, c_int64, c_int, c_int64, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                           c_float, c_float, P],
+        "gllm_moe_route_align": [P, c_int64, c_int, c_int64, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                 c_int, c_float, c_float, P, P, P, P, c_int, c_int, P],
         "gllm_moe_align": [P, P, P, P, P, c_int, c_int, c_int, c_int, P],
         "gllm_moe_gemm_{t}": [P, c_int64, c_int, P, c_int64, c_int64, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P,
                               c_float, c_float, c_float, P],
-        "gllm_moe_combine_{t}": [P, P, P, P, P, c_int, c_int, c_int, P, c_int64, P],
+        "gllm_moe_combine_{t}": [P, c_int, c_int64, P, P, P, P, c_int, c_int, c_int, P, c_int64, P],
         "gllm_moe_relu_sq_bf16": [P, P, c_int64, P],
         "gllm_moe_gather_{t}": [P, c_int64, P, P, c_int, c_int, c_int, P, P, P],
     },
@@ -361,9 +365,25 @@ class _Added:
 ADDED = _Added()
 
 
+class RowSum:
+    """The result of routed experts that has not been added up per token: ``y [parts, rows, width]`` (fp32; the parts are
+    added first), of which token ``t``'s row is the sum over its ``top`` slots of rows ``row_of_pair[t * top + s]``
+    (without ``row_of_pair``: ``t * top + s``), times ``weights [tokens, top]`` when given.  The kernel that norms and
+    adds a sublayer's result (``add_cast``, ``add_rmsnorm`` of a ``Pending``) takes it as it is."""
+
+    def __init__(self, y: torch.Tensor, row_of_pair, weights, tokens: int, top: int, dtype: torch.dtype):
+        self.y, self.row_of_pair, self.weights, self.top, self.dtype = y, row_of_pair, weights, int(top), dtype
+        self.shape = (int(tokens), y.shape[-1])
+
+    def tensor(self) -> torch.Tensor:
+        from gllm_b200.ops import moe
+
+        return moe.combine(self.y, self.weights, None, self.dtype, self.row_of_pair, tokens=self.shape[0], top=self.top)
+
+
 def as_tensor(x):
-    """``x`` itself, or the summed tensor of a SplitSum."""
-    return x.tensor() if isinstance(x, SplitSum) else x
+    """``x`` itself, or the summed tensor of a SplitSum (or a RowSum)."""
+    return x.tensor() if isinstance(x, (SplitSum, RowSum)) else x
 
 
 class Pending:
@@ -566,7 +586,14 @@ def _pending_add_rmsnorm(pending: Pending, resid, weight, eps, out_dtype, rows, 
     n_total, hidden = resid.numel() // resid.shape[-1], resid.shape[-1]
     value = pending.value
     parts_ptr, n_parts, part_stride = _parts_args(value)
-    if isinstance(value, SplitSum):
+    row_sum = (None, 0, 0, None, None, 0)
+    if isinstance(value, RowSum):
+        if tuple(value.shape) != tuple(resid.shape) or value.dtype != out_dtype:
+            raise ValueError("the pending rows and the residual differ in shape or dtype")
+        row_sum = (value.y.data_ptr(), value.y.shape[0], value.y.stride(0), _ptr(value.row_of_pair), _ptr(value.weights),
+                   value.top)
+        value = None
+    elif isinstance(value, SplitSum):
         if tuple(value.shape) != tuple(resid.shape) or value.dtype != out_dtype:
             raise ValueError("the pending value and the residual differ in shape or dtype")
         value = None
@@ -592,7 +619,7 @@ def _pending_add_rmsnorm(pending: Pending, resid, weight, eps, out_dtype, rows, 
     f = _fn("postnorm", f"gllm_postnorm_add_rmsnorm_{_suffix(out_dtype)}")
     _check(f(_ptr(value), parts_ptr, n_parts, part_stride, _ptr(pending.post_weight), pending.post_eps,
              _ptr(pending.extra), resid.data_ptr(), _ptr(weight), float(eps), out.data_ptr(), _ptr(rows), n_rows,
-             hidden, _stream()), "postnorm_add_rmsnorm")
+             hidden, *row_sum, _stream()), "postnorm_add_rmsnorm")
     return out
 
 

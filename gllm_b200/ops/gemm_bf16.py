@@ -62,28 +62,32 @@ _grouped = None
 
 def linear_grouped(x: torch.Tensor, weight: torch.Tensor, group_of_tile: torch.Tensor, num_tiles: torch.Tensor,
                    gated: bool, wide: bool, act: tuple = (1.0, 0.0, 0.0),
-                   row_scale: torch.Tensor | None = None) -> torch.Tensor:
+                   row_scale: torch.Tensor | None = None, tile_rows: int = 128, splits: int = 1) -> torch.Tensor:
     """``out[r] = x[r] @ weight[g(r)].T`` on the tcgen05 kernel, the rows of ``x [rows, k]`` (bf16, ``rows`` a
-    multiple of 128) coming in tiles of 128 that each belong to one group: ``group_of_tile [rows / 128]`` and
+    multiple of ``tile_rows``: 128, or 16, 32 or 64, for which the weight is the 128-row operand) coming in tiles of
+    ``tile_rows`` that each belong to one group: ``group_of_tile [rows / tile_rows]`` and
     ``num_tiles [1]`` (int32, on the device; tiles behind ``num_tiles`` are neither read nor written).  ``weight
     [groups, n, k]``; ``gated``: every group's rows are stacked by ``interleave_gate_up`` and the result is bf16
     ``silu(gate) * up`` ``[rows, n / 2]`` (or what ``act``, the slope, limit and offset of ``linear_gated``, says, of
-    gate and up products that are multiplied by the row's number of ``row_scale`` first); otherwise fp32 ``[rows, n]``.  ``wide``: tiles of 256 weight rows (many
+    gate and up products that are multiplied by the row's number of ``row_scale`` first); otherwise fp32 ``[rows, n]``, or with ``splits`` > 1 (small tiles) ``[splits, rows, n]``, one unsummed part per range
+    of k.  ``wide``: tiles of 256 weight rows (many
     rows per group) instead of 128."""
     global _grouped
     if _grouped is None:
         f = load_module("gemm_bf16").gllm_gemm_bf16_grouped
-        f.argtypes = [P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, c_int, P, c_float, c_float, c_float, P, P]
+        f.argtypes = [P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, c_int, P, c_float, c_float, c_float, c_int, c_int,
+                      P, P]
         f.restype = c_int
         _grouped = f
     from gllm_b200.ops import _check, _ptr, _stream, status_word
 
     rows, k = x.shape
     groups, n, _ = weight.shape
-    out = torch.empty((rows, n // 2 if gated else n), dtype=torch.bfloat16 if gated else torch.float32, device=x.device)
+    shape = (rows, n // 2) if gated else (rows, n) if splits == 1 else (splits, rows, n)
+    out = torch.empty(shape, dtype=torch.bfloat16 if gated else torch.float32, device=x.device)
     _check(_grouped(x.data_ptr(), weight.data_ptr(), out.data_ptr(), int(gated), rows, n, k, groups,
                     group_of_tile.data_ptr(), num_tiles.data_ptr(), int(wide), _ptr(row_scale), *act,
-                    status_word(x.device).data_ptr(), _stream()), "linear_grouped")
+                    int(tile_rows), int(splits), status_word(x.device).data_ptr(), _stream()), "linear_grouped")
     return out
 
 

@@ -6,38 +6,59 @@ from __future__ import annotations
 
 import torch
 
-from gllm_b200.ops import _check, _cuda, _fn, _ptr, _stream, _suffix
+from gllm_b200.ops import RowSum, SplitSum, _check, _cuda, _fn, _parts_args, _ptr, _stream, _suffix
 
 TILE_ROWS = 16        # rows of one tile of the expert products: an expert's pairs are padded to a multiple of it
 PLAIN_GATE = (1.0, 0.0, 0.0)    # slope, limit, offset of a gated expert's activation: silu(gate) * up
 TENSOR_CORE_TILE_ROWS = 128     # the same for the tcgen05 products (the rows of one accumulator tile)
 
 
-def route(logits: torch.Tensor, correction: torch.Tensor | None, top: int, groups: int = 1, groups_kept: int = 1,
-          renormalize: bool = False, score: str = "sigmoid", group_score: str = "top2", renormalize_eps: float = 0.0,
-          scale: float = 1.0):
-    """From fp32 router logits ``[n, experts]`` to the chosen experts ``[n, top]`` int32 and their weights fp32.
-    Scores ``s = sigmoid(logits)`` (``score`` "softmax": the softmax over all experts); the choice is made on
-    ``s + correction`` among the experts of the ``groups_kept`` best of ``groups`` equal groups of neighbours (a
-    group's score: the sum of its two largest choice scores, with ``group_score`` "max" its largest); the weights are
-    the chosen ``s``, divided by their sum (plus ``renormalize_eps``) with ``renormalize``, times ``scale``."""
-    if score not in ("sigmoid", "softmax") or group_score not in ("top2", "max"):
-        raise ValueError("router scores are 'sigmoid' or 'softmax', group scores 'top2' or 'max'")
+def _router_args(logits):
+    """(pointer, row stride, parts, part stride, tokens, experts) of fp32 router logits: a tensor or a SplitSum."""
+    if isinstance(logits, SplitSum):
+        ptr, n_parts, part_stride = _parts_args(logits)
+        if logits.dtype != torch.float32:
+            raise TypeError("router logits are fp32")
+        return ptr, logits.shape[1], n_parts, part_stride, *logits.shape
     _cuda(logits, "logits", torch.float32, contiguous=False)
     if logits.dim() != 2 or logits.stride(1) != 1:
         raise ValueError("router logits must be [tokens, experts] with contiguous columns")
+    return logits.data_ptr(), logits.stride(0), 0, 0, *logits.shape
+
+
+def _rule_args(correction, experts, top, groups, groups_kept, renormalize, score, group_score, renormalize_eps, scale):
+    if score not in ("sigmoid", "softmax") or group_score not in ("top2", "max"):
+        raise ValueError("router scores are 'sigmoid' or 'softmax', group scores 'top2' or 'max'")
     if correction is not None:
         _cuda(correction, "correction", torch.float32)
-        if correction.numel() != logits.shape[1]:
+        if correction.numel() != experts:
             raise ValueError("one correction value per expert is needed")
-    n, experts = logits.shape
+    return (experts, int(top), int(groups), int(groups_kept), int(renormalize), int(score == "softmax"),
+            int(group_score == "max"), float(renormalize_eps), float(scale))
+
+
+def route(logits, correction: torch.Tensor | None, top: int, groups: int = 1, groups_kept: int = 1,
+          renormalize: bool = False, score: str = "sigmoid", group_score: str = "top2", renormalize_eps: float = 0.0,
+          scale: float = 1.0):
+    """From fp32 router logits ``[n, experts]`` (a tensor or a SplitSum) to the chosen experts ``[n, top]`` int32 and their
+    weights fp32.  Scores ``s = sigmoid(logits)`` (``score`` "softmax": the softmax over all experts); the choice is made
+    on ``s + correction`` among the experts of the ``groups_kept`` best of ``groups`` equal groups of neighbours (a
+    group's score: the sum of its two largest choice scores, with ``group_score`` "max" its largest); the weights are
+    the chosen ``s``, divided by their sum (plus ``renormalize_eps``) with ``renormalize``, times ``scale``."""
+    ptr, stride, n_parts, part_stride, n, experts = _router_args(logits)
+    rule = _rule_args(correction, experts, top, groups, groups_kept, renormalize, score, group_score, renormalize_eps, scale)
     ids = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
-    _check(_fn("moe", "gllm_moe_route")(logits.data_ptr(), logits.stride(0), _ptr(correction), ids.data_ptr(),
-                                        weights.data_ptr(), n, experts, int(top), int(groups), int(groups_kept),
-                                        int(renormalize), int(score == "softmax"), int(group_score == "max"),
-                                        float(renormalize_eps), float(scale), _stream()), "moe_route")
+    _check(_fn("moe", "gllm_moe_route")(ptr, stride, n_parts, part_stride, _ptr(correction), ids.data_ptr(),
+                                        weights.data_ptr(), n, *rule, _stream()), "moe_route")
     return ids, weights
+
+
+def _plan_tensors(pairs: int, experts: int, tile_rows: int, want_sorted: bool, want_rows: bool, device):
+    max_tiles = -(-pairs // tile_rows) + min(experts, pairs)
+    i32 = lambda n: torch.empty(n, dtype=torch.int32, device=device)
+    return (i32(max_tiles * tile_rows) if want_sorted else None, i32(max_tiles), i32(1),
+            i32(pairs) if want_rows else None)
 
 
 def align(ids: torch.Tensor, experts: int, tile_rows: int = TILE_ROWS, want_rows: bool = False):
@@ -46,17 +67,35 @@ def align(ids: torch.Tensor, experts: int, tile_rows: int = TILE_ROWS, want_rows
     ``want_rows`` also ``row_of_pair [pairs]``, the row each pair got."""
     _cuda(ids, "ids", torch.int32)
     pairs = ids.numel()
-    max_tiles = -(-pairs // tile_rows) + min(experts, pairs)
-    sorted_pairs = torch.empty(max_tiles * tile_rows, dtype=torch.int32, device=ids.device)
-    tile_expert = torch.empty(max_tiles, dtype=torch.int32, device=ids.device)
-    num_tiles = torch.empty(1, dtype=torch.int32, device=ids.device)
-    row_of_pair = torch.empty(pairs, dtype=torch.int32, device=ids.device) if want_rows else None
-    _check(_fn("moe", "gllm_moe_align")(ids.data_ptr(), sorted_pairs.data_ptr(), tile_expert.data_ptr(),
-                                        num_tiles.data_ptr(), _ptr(row_of_pair), pairs, int(experts), int(tile_rows),
-                                        max_tiles, _stream()), "moe_align")
-    if want_rows:
-        return sorted_pairs, tile_expert, num_tiles, row_of_pair
-    return sorted_pairs, tile_expert, num_tiles
+    plan = _plan_tensors(pairs, experts, tile_rows, True, want_rows, ids.device)
+    _check(_fn("moe", "gllm_moe_align")(ids.data_ptr(), *(_ptr(t) for t in plan), pairs, int(experts), int(tile_rows),
+                                        plan[1].numel(), _stream()), "moe_align")
+    return plan if want_rows else plan[:3]
+
+
+# most tokens whose routing and sorting one block does in one launch
+ROUTE_ALIGN_TOKENS = 64
+
+
+def route_and_align(logits, correction, top: int, tile_rows: int, want_sorted: bool, want_rows: bool, groups: int = 1,
+                    groups_kept: int = 1, renormalize: bool = False, score: str = "sigmoid", group_score: str = "top2",
+                    renormalize_eps: float = 0.0, scale: float = 1.0):
+    """``route`` and ``align`` one after the other, in one launch for up to ``ROUTE_ALIGN_TOKENS`` tokens: ``(ids, weights,
+    (sorted | None, tile_expert, num_tiles, row_of_pair | None))``."""
+    ptr, stride, n_parts, part_stride, n, experts = _router_args(logits)
+    if n > ROUTE_ALIGN_TOKENS or 32 * (2 * experts + groups) * 4 + (3 * experts + 1) * 4 > 48 * 1024:
+        ids, weights = route(logits, correction, top, groups, groups_kept, renormalize, score, group_score,
+                             renormalize_eps, scale)
+        plan = align(ids, experts, tile_rows, want_rows=True)
+        return ids, weights, plan
+    rule = _rule_args(correction, experts, top, groups, groups_kept, renormalize, score, group_score, renormalize_eps, scale)
+    ids = torch.empty((n, top), dtype=torch.int32, device=logits.device)
+    weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    plan = _plan_tensors(n * top, experts, tile_rows, want_sorted, want_rows, logits.device)
+    _check(_fn("moe", "gllm_moe_route_align")(ptr, stride, n_parts, part_stride, _ptr(correction), ids.data_ptr(),
+                                              weights.data_ptr(), n, *rule, *(_ptr(t) for t in plan), int(tile_rows),
+                                              plan[1].numel(), _stream()), "moe_route_align")
+    return ids, weights, plan
 
 
 def gather_rows(x: torch.Tensor, top: int, row_of_pair: torch.Tensor, rows: int, weights: torch.Tensor | None = None):
@@ -110,20 +149,22 @@ def expert_product(a: torch.Tensor, rows_per_input: int, weight: torch.Tensor, p
     return out
 
 
-def combine(y: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None, out_dtype: torch.dtype,
-            row_of_pair: torch.Tensor | None = None, shared_gate: torch.Tensor | None = None,
-            weighted: bool = True) -> torch.Tensor:
-    """``out[t] = sum_s weights[t, s] * y[t * top + s] (+ shared[t])``, summed in slot order in fp32 (``weighted``
-    False: without the weights, which the experts' inputs had); with
+def combine(y: torch.Tensor, weights: torch.Tensor | None, shared: torch.Tensor | None, out_dtype: torch.dtype,
+            row_of_pair: torch.Tensor | None = None, shared_gate: torch.Tensor | None = None, tokens: int | None = None,
+            top: int | None = None) -> torch.Tensor:
+    """``out[t] = sum_s weights[t, s] * y[t * top + s] (+ shared[t])``, summed in slot order in fp32 (``weights`` None: 1
+    each; ``tokens`` and ``top`` are then named); ``y`` may be ``[parts, rows, width]``, the parts being added first; with
     ``row_of_pair`` the pair's result is row ``row_of_pair[t * top + s]`` of ``y``; with ``shared_gate`` (fp32, one
     logit per token; may be a column of a wider matrix) the shared result is multiplied by its sigmoid."""
     _cuda(y, "y", torch.float32)
-    _cuda(weights, "weights", torch.float32)
-    n, top = weights.shape
-    width = y.shape[1]
+    y = y if y.dim() == 3 else y[None]
+    if weights is not None:
+        _cuda(weights, "weights", torch.float32)
+        tokens, top = weights.shape
+    n, width = int(tokens), y.shape[2]
     if row_of_pair is not None:
         _cuda(row_of_pair, "row_of_pair", torch.int32)
-    if (y.shape[0] != n * top and row_of_pair is None) or (row_of_pair is not None and row_of_pair.numel() != n * top):
+    if (y.shape[1] != n * top and row_of_pair is None) or (row_of_pair is not None and row_of_pair.numel() != n * top):
         raise ValueError("one result row per (token, slot) pair is needed")
     if shared is not None:
         _cuda(shared, "shared", out_dtype)
@@ -136,10 +177,10 @@ def combine(y: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None,
             raise ValueError("the shared expert's gate is one logit per token")
         gate_stride = shared_gate.stride(0)
     out = torch.empty((n, width), dtype=out_dtype, device=y.device)
-    _check(_fn("moe", f"gllm_moe_combine_{_suffix(out_dtype)}")(y.data_ptr(),
-                                                               weights.data_ptr() if weighted else None, _ptr(shared),
-                                                               out.data_ptr(), _ptr(row_of_pair), n, top, width,
-                                                               _ptr(shared_gate), gate_stride, _stream()), "moe_combine")
+    _check(_fn("moe", f"gllm_moe_combine_{_suffix(out_dtype)}")(y.data_ptr(), y.shape[0], y.stride(0), _ptr(weights),
+                                                               _ptr(shared), out.data_ptr(), _ptr(row_of_pair), n,
+                                                               int(top), width, _ptr(shared_gate), gate_stride,
+                                                               _stream()), "moe_combine")
     return out
 
 
@@ -152,10 +193,52 @@ def relu_squared_rows(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def grouped_tile_rows(pairs: int, experts: int) -> int:
+    """Rows of a tile of the tensor-core products: small tiles (the weight is then the 128-row operand, and a tile's rows
+    cost little) while an expert gets few rows on average."""
+    per_expert = pairs / experts
+    return 16 if per_expert <= 8 else 32 if per_expert <= 20 else 64 if per_expert <= 40 else TENSOR_CORE_TILE_ROWS
+
+
+def _down_splits(pairs: int, experts: int, rows: int, k: int, device) -> int:
+    """Ranges of K the second product is cut into when its tiles alone would leave most SMs without work."""
+    tiles = min(pairs, experts) * -(-rows // 128)
+    sms = torch.cuda.get_device_properties(device).multi_processor_count
+    blocks = -(-k // 64)
+    best = 1
+    for s in range(2, 5):
+        if tiles * s <= sms and blocks // s >= 4 and -(-blocks // s) * (s - 1) < blocks:
+            best = s
+    return best
+
+
+class Choice:
+    """Which experts serve which tokens: ids and weights ``[n, top]`` and the (token, slot) pairs sorted by expert."""
+
+    def __init__(self, ids, weights, plan, tile_rows: int):
+        self.ids, self.weights, self.plan, self.tile_rows = ids, weights, plan, tile_rows
+
+
+def choose(logits, correction, top: int, tensor_cores: bool, **rule) -> Choice:
+    """Route and sort for ``apply_choice`` (``rule``: the options of ``route``)."""
+    n, experts = logits.shape
+    tile = grouped_tile_rows(n * top, experts) if tensor_cores else TILE_ROWS
+    return Choice(*route_and_align(logits, correction, top, tile, want_sorted=not tensor_cores, want_rows=tensor_cores, **rule),
+                  tile)
+
+
 def apply_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
-                  w_down: torch.Tensor, shared: torch.Tensor | None, tensor_cores: bool, gated: bool = True,
-                  shared_gate: torch.Tensor | None = None, act: tuple = PLAIN_GATE,
-                  weight_on_input: bool = False) -> torch.Tensor:
+                  w_down: torch.Tensor, shared: torch.Tensor | None, tensor_cores: bool, **options) -> torch.Tensor:
+    """``apply_choice`` for a choice that is already made: ``ids`` and ``weights`` ``[n, top]``."""
+    tile = grouped_tile_rows(ids.numel(), w_gate_up.shape[0]) if tensor_cores else TILE_ROWS
+    plan = align(ids, w_gate_up.shape[0], tile, want_rows=True)
+    return apply_choice(x, Choice(ids, weights, plan, tile), w_gate_up, w_down, shared, tensor_cores, **options)
+
+
+def apply_choice(x: torch.Tensor, choice: Choice, w_gate_up: torch.Tensor, w_down: torch.Tensor,
+                 shared: torch.Tensor | None, tensor_cores: bool, gated: bool = True,
+                 shared_gate: torch.Tensor | None = None, act: tuple = PLAIN_GATE, weight_on_input: bool = False,
+                 defer_sum: bool = False):
     """``out[t] = sum_s weights[t, s] * expert_{ids[t, s]}(x[t]) (+ shared[t])`` with ``expert_e(x) = w_down[e]
     (silu(gate) * up)``.  ``tensor_cores``: ``w_gate_up [experts, 2 * ff, width]`` is stacked per expert by
     ``interleave_gate_up``; the tokens' rows are copied into the order of the sorted pairs, both products read and
@@ -164,28 +247,36 @@ def apply_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_g
     experts without a gate, ``expert_e(x) = w_down[e] relu(w_up[e] x)^2`` with ``w_gate_up [experts, ff, width]`` the
     up weights.  ``shared_gate``: see ``combine``.  ``act``: the slope, limit and offset of the gated activation.
     ``weight_on_input``: ``out[t] = sum_s expert(weights[t, s] * x[t])`` instead; the weight is applied to the first
-    product's fp32 sums, which is the same and spares a rounding."""
-    experts, (_, top), pairs = w_gate_up.shape[0], ids.shape, ids.numel()
+    product's fp32 sums, which is the same and spares a rounding.  ``defer_sum`` (without a shared expert): the pairs'
+    results are returned as an ``ops.RowSum``, for a kernel that adds them up itself."""
+    experts, (n, top), pairs = w_gate_up.shape[0], choice.ids.shape, choice.ids.numel()
+    weights, (sorted_pairs, tile_expert, num_tiles, row_of_pair) = choice.weights, choice.plan
     if not tensor_cores:
-        plan = align(ids, experts)
+        plan, row_of_pair = (sorted_pairs, tile_expert, num_tiles), None
         hidden = expert_product(x, top, w_gate_up, plan, pairs, gated=gated, relu_squared=not gated, act=act,
                                 row_scale=weights if weight_on_input else None)
         y = expert_product(hidden, 1, w_down, plan, pairs, gated=False)
-        return combine(y, weights, shared, x.dtype, shared_gate=shared_gate, weighted=not weight_on_input)
-    from gllm_b200.ops import gemm_bf16
-
-    _, tile_expert, num_tiles, row_of_pair = align(ids, experts, TENSOR_CORE_TILE_ROWS, want_rows=True)
-    wide = pairs > 2048
-    rows, row_scale = tile_expert.numel() * TENSOR_CORE_TILE_ROWS, None
-    if weight_on_input:
-        if not gated:
-            raise ValueError("weights on the input of the tensor-core products are for gated experts")
-        xs, row_scale = gather_rows(x, top, row_of_pair, rows, weights)
     else:
-        xs = gather_rows(x, top, row_of_pair, rows)
-    hidden = gemm_bf16.linear_grouped(xs, w_gate_up, tile_expert, num_tiles, gated=gated, wide=wide, act=act,
-                                      row_scale=row_scale)
-    if not gated:
-        hidden = relu_squared_rows(hidden)
-    y = gemm_bf16.linear_grouped(hidden, w_down, tile_expert, num_tiles, gated=False, wide=wide)
-    return combine(y, weights, shared, x.dtype, row_of_pair, shared_gate=shared_gate, weighted=not weight_on_input)
+        from gllm_b200.ops import gemm_bf16
+
+        wide = pairs > 2048
+        rows, row_scale = tile_expert.numel() * choice.tile_rows, None
+        if weight_on_input:
+            if not gated:
+                raise ValueError("weights on the input of the tensor-core products are for gated experts")
+            xs, row_scale = gather_rows(x, top, row_of_pair, rows, weights)
+        else:
+            xs = gather_rows(x, top, row_of_pair, rows)
+        hidden = gemm_bf16.linear_grouped(xs, w_gate_up, tile_expert, num_tiles, gated=gated, wide=wide, act=act,
+                                          row_scale=row_scale, tile_rows=choice.tile_rows)
+        if not gated:
+            hidden = relu_squared_rows(hidden)
+        splits = 1
+        if choice.tile_rows != TENSOR_CORE_TILE_ROWS:
+            splits = _down_splits(pairs, experts, w_down.shape[1], w_down.shape[2], x.device)
+        y = gemm_bf16.linear_grouped(hidden, w_down, tile_expert, num_tiles, gated=False, wide=wide,
+                                     tile_rows=choice.tile_rows, splits=splits)
+    weights = None if weight_on_input else weights
+    if defer_sum and shared is None:
+        return RowSum(y if y.dim() == 3 else y[None], row_of_pair, weights, n, top, x.dtype)
+    return combine(y, weights, shared, x.dtype, row_of_pair, shared_gate=shared_gate, tokens=n, top=top)

@@ -168,6 +168,9 @@ class StepContext:
     # Set by a block around a part's call: the part may leave its last product's bias to the block's next kernel and
     # return ``ops.Biased(value, bias)``.
     takes_bias: bool = False
+    # Set by a block around a part's call: the part may leave the sum over its experts to the block's next kernel and
+    # return an ``ops.RowSum``.
+    takes_row_sum: bool = False
     # what a layer leaves for later layers of the same step (key -> tensor over the step's tokens)
     shared: dict = field(default_factory=dict)
     # fp32 [plan entries + 1, n, hidden] of a model that averages over its depth: the embedding output, then every

@@ -75,7 +75,9 @@ class ResultOnlyNormBlock(Block):
         out = self.mixer_norm.pending(self.mixer.forward(x, ctx, cache))
         if self.feed_forward is not None:
             x = ops.add_cast(out, resid, ctx.dtype)
+            ctx.takes_row_sum = True
             out = self.feed_forward_norm.pending(self.feed_forward.forward(x, ctx))
+            ctx.takes_row_sum = False
         return out, resid
 
 

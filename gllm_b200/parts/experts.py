@@ -7,7 +7,7 @@ best of ``groups`` equal groups of neighbouring experts, a group's score being t
 scores.  The result is ``sum_e s_e * expert_e(x)`` over the chosen experts (weights divided by their sum with
 ``renormalize``) plus the shared expert's.  The (token, expert) pairs are sorted by expert on the device and the
 experts' products run over tiles of one expert each: in bf16, with sizes it takes, on the tcgen05 kernel of the dense
-products in its grouped form (tiles of 128 rows, ``csrc/gemm_bf16.cu``), otherwise on a CUDA-core kernel (tiles of
+products in its grouped form (tiles of 128 rows, or of 16 to 64 while an expert gets few, ``csrc/gemm_bf16.cu``), otherwise on a CUDA-core kernel (tiles of
 16 rows, ``csrc/moe.cu``); nothing about the choice reaches the host.
 
 Options for other designs: ``score`` "softmax" (scores are the softmax of the logits over all experts);
@@ -120,15 +120,17 @@ class RoutedExperts(FeedForward):
             self.shared.load(get, dtype, device)
 
     def forward(self, x, ctx):
-        logits = ops.linear(x, self.w_router, out_dtype=torch.float32)
+        logits = ops.linear(x, self.w_router, out_dtype=torch.float32, split_ok=not self.has_shared_gate)
         gate = logits[:, self.experts] if self.has_shared_gate else None
-        ids, weights = moe.route(logits[:, : self.experts], self.correction, self.top, self.groups, self.groups_kept,
-                                 self.renormalize, score=self.score, group_score=self.group_score,
-                                 renormalize_eps=self.renormalize_eps, scale=self.scale)
+        choice = moe.choose(logits[:, : self.experts] if self.has_shared_gate else logits, self.correction, self.top,
+                            self.tensor_cores, groups=self.groups, groups_kept=self.groups_kept,
+                            renormalize=self.renormalize, score=self.score, group_score=self.group_score,
+                            renormalize_eps=self.renormalize_eps, scale=self.scale)
         shared = None
         if self.shared is not None:
             sink, ctx.residual_sink = getattr(ctx, "residual_sink", None), None
             shared = ops.as_tensor(self.shared.forward(x, ctx))
             ctx.residual_sink = sink
-        return moe.apply_experts(x, ids, weights, self.w_gate_up, self.w_down, shared, self.tensor_cores,
-                                 gated=self.gated, shared_gate=gate, act=self.act, weight_on_input=self.weight_on_input)
+        return moe.apply_choice(x, choice, self.w_gate_up, self.w_down, shared, self.tensor_cores, gated=self.gated,
+                                shared_gate=gate, act=self.act, weight_on_input=self.weight_on_input,
+                                defer_sum=getattr(ctx, "takes_row_sum", False))

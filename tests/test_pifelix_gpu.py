@@ -277,7 +277,9 @@ def test_norm_of_a_result_and_the_residual_as_it_is(dtype, rows, width):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("n,width,ff,experts,top,limit", [(37, 64, 64, 8, 2, 0.5), (1, 44, 20, 4, 1, 1.0), (300, 128, 64, 16, 4, 0.3),
-                                                         (9, 48, 24, 6, 6, 2.0), (1500, 256, 128, 4, 2, 0.7), (130, 64, 192, 3, 1, 0.4)])
+                                                         (9, 48, 24, 6, 6, 2.0), (1500, 256, 128, 4, 2, 0.7), (130, 64, 192, 3, 1, 0.4),
+                                                         (3, 64, 1024, 4, 2, 0.6), (100, 128, 64, 8, 2, 0.5),
+                                                         (60, 200, 320, 6, 2, 0.5), (2, 136, 576, 9, 3, 1.1)])
 def test_experts_with_weights_on_their_inputs_and_a_clamped_gate(dtype, n, width, ff, experts, top, limit):
     """``sum_s expert(w_s x)``: bf16 sizes that the tensor-core kernel takes run there, the others (and float32) on the
     CUDA cores.  The clamps bite, and the weights on the output, or no clamps, would give another result."""
@@ -313,8 +315,60 @@ def test_experts_with_weights_on_their_inputs_and_a_clamped_gate(dtype, n, width
                             act=(1.702, limit, 1.0), weight_on_input=True).double().cpu()
     tol = (1e-5 if dtype == torch.float32 else 1e-2) * max(1.0, float(want.abs().max()))
     assert float((got - want).abs().max()) <= tol
+    # the sum over the experts left to the kernel that norms and adds the result
+    tile = moe.grouped_tile_rows(n * top, experts) if cores else moe.TILE_ROWS
+    choice = moe.Choice(ids.cuda(), wts.cuda(), moe.align(ids.cuda(), experts, tile, want_rows=True), tile)
+    rows = moe.apply_choice(x.to(dtype).cuda(), choice, w_gu, wd.to(dtype).cuda().contiguous(), None, cores,
+                            act=(1.702, limit, 1.0), weight_on_input=True, defer_sum=True)
+    assert isinstance(rows, ops.RowSum) and tuple(rows.shape) == (n, width)
+    assert not (cores and n == 3) or rows.y.shape[0] > 1              # few tiles: the second product is cut along K
+    assert float((ops.as_tensor(rows).double().cpu() - want).abs().max()) <= tol
+    resid, w = torch.randn(n, width, generator=g) * 3, torch.randn(width, generator=g)
+    for weights, value in ((None, got.cpu()), (wts, None)):
+        if weights is not None:                                       # a sum with weights: the same rows, weighted
+            rows = ops.RowSum(rows.y, rows.row_of_pair, wts.cuda(), n, top, dtype)
+            value = ops.as_tensor(rows).double().cpu()
+        r = resid.cuda()
+        cast = ops.add_cast(ops.Pending(rows, w.cuda(), 1e-3), r, dtype)
+        total = resid.double() + plain.rms(value, w.double(), 1e-3)
+        assert torch.allclose(r.double().cpu(), total, atol=1e-4 if dtype == torch.float32 else 2e-2)
+        assert torch.equal(cast, r.to(dtype))
+        pick = torch.tensor([n - 1, 0], dtype=torch.int32)
+        normed = ops.add_rmsnorm(ops.Pending(rows, w.cuda(), 1e-3), resid.cuda(), w.cuda(), 1e-5, dtype, rows=pick.cuda())
+        want_rows = plain.rms(total, w.double(), 1e-5)[pick.long()]
+        assert torch.allclose(normed.double().cpu(), want_rows, atol=1e-4 if dtype == torch.float32 else 5e-2, rtol=1e-2)
     for other in (reference(None), reference(limit, on_input=False)):
         assert n < 9 or float((other - want).abs().max()) > 5 * tol
+
+
+@pytest.mark.parametrize("n,experts,top,splits", [(1, 8, 2, 0), (7, 3, 1, 4), (64, 40, 5, 2), (65, 16, 4, 3), (40, 5, 5, 0)])
+def test_routing_and_sorting_in_one_launch(n, experts, top, splits):
+    """Scores, choice, weights and the sort of the pairs by expert, the logits as a tensor or as unsummed splits of the
+    router's product, for few tokens (one launch) and more (two)."""
+    from gllm_b200 import ops
+    from gllm_b200.ops import moe
+
+    g = torch.Generator().manual_seed(n + experts)
+    parts = torch.randn(max(splits, 1), n, experts, generator=g)
+    z = parts.sum(0)
+    logits = ops.SplitSum(parts.cuda(), torch.float32) if splits else z.cuda()
+    for cores in (False, True):
+        choice = moe.choose(logits, None, top, cores)
+        order = torch.sort(z.double(), dim=-1, descending=True, stable=True).indices[:, :top]
+        assert torch.equal(choice.ids.long().cpu(), order)
+        want = plain.sigmoid(z.double()).gather(1, order)
+        assert torch.allclose(choice.weights.double().cpu(), want, atol=1e-6)
+        sorted_pairs, tile_expert, num_tiles, row_of_pair = (t if t is None else t.cpu() for t in choice.plan)
+        ids, tile = choice.ids.reshape(-1).cpu(), choice.tile_rows
+        counts = torch.bincount(ids.long(), minlength=experts)
+        assert int(num_tiles) == int(((counts + tile - 1) // tile).sum())
+        if cores:
+            assert len(set(row_of_pair.tolist())) == n * top
+            assert all(int(tile_expert[int(row) // tile]) == int(e) for row, e in zip(row_of_pair, ids))
+        else:
+            for row, p in enumerate(sorted_pairs[: int(num_tiles) * tile].tolist()):
+                assert p < 0 or int(ids[p]) == int(tile_expert[row // tile])
+            assert sorted(p for p in sorted_pairs.tolist() if p >= 0) == list(range(n * top))
 
 
 # ------------------------------------------------------------------ each mechanism alone in a model of one layer
