@@ -344,7 +344,7 @@ int conv_qkv_launch(const ConvQkv<T>& a, int num_requests, int max_q_len, cudaSt
   const int keep = a.taps - 1, pairs4 = a.inv_freq ? (a.rotary_dim / 2 + 3) & ~3 : 0;
   const int64_t places = (int64_t)gllm_sm_count() * GLLM_CONV_QKV_BLOCKS / ((int64_t)num_requests * groups);
   int run = (int)((max_q_len + (places > 1 ? places : 1) - 1) / (places > 1 ? places : 1));
-  run = std::min((std::max(run, 4) + 1) & ~1, pairs4 > 80 ? 40 : 64);
+  run = std::min((std::max(run, 4) + 1) & ~1, std::min(256, 40 * 1024 / (8 * pairs4 + 4)));
   if (run < keep) run = keep;
   auto misaligned = [](const void* p) { return p != nullptr && (reinterpret_cast<uintptr_t>(p) & 15) != 0; };
   const bool vec = a.dk % CQ_COLS == 0 && a.dv % CQ_COLS == 0 && (a.proj == nullptr || a.stride % CQ_COLS == 0) &&

@@ -84,7 +84,7 @@ def attention_decode(batch=64, context=2048, hq=32, hkv=8, d=64, block_size=16, 
 
 
 def attention_prefill(tokens=2048, context=0, hq=32, hkv=8, d=64, block_size=16, iters=5, peaks=None, tmem=1,
-                      chunk=0):
+                      chunk=0, window=0):
     from gllm_b200.ops import attention_bf16
 
     pool, table = _paged_cache(1, context + tokens, hkv, d, block_size)
@@ -95,15 +95,16 @@ def attention_prefill(tokens=2048, context=0, hq=32, hkv=8, d=64, block_size=16,
     out = torch.empty(tokens, hq * d, dtype=torch.bfloat16, device="cuda")
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
     kernel = attention_bf16.prefill_attention_tmem if tmem else attention_bf16.prefill_attention
-    fn = lambda: kernel(qkv, qkv.shape[1], pool, table, cu, ctx, slots, 1, tokens, hq, 1.0 / math.sqrt(d), -chunk, out)
+    fn = lambda: kernel(qkv, qkv.shape[1], pool, table, cu, ctx, slots, 1, tokens, hq, 1.0 / math.sqrt(d), window or -chunk, out)
     us = _time(fn, iters, flush)
     pairs = (sum(p % chunk + 1 for p in range(context, context + tokens)) if chunk
-             else tokens * context + tokens * (tokens + 1) / 2)
+             else _visible(tokens, context, window))
     flops = 4.0 * d * hq * pairs
     tf = flops / us / 1e6
     return {"kernel": "attention_prefill (tcgen05)" if tmem else "attention_prefill (mma.sync)", "us": round(us, 2), "flops": flops, "achieved_tflops": round(tf, 1),
             "frac_of_bf16_peak": round(tf / peaks["bf16_tflops"], 4),
-            "shape": dict(tokens=tokens, context=context, heads=hq, kv_heads=hkv, head_dim=d, block_size=block_size, chunk=chunk)}
+            "shape": dict(tokens=tokens, context=context, heads=hq, kv_heads=hkv, head_dim=d, block_size=block_size, chunk=chunk,
+                          window=window)}
 
 
 def linear(m=8, n=16384, k=2048, iters=5, peaks=None, out_fp32=False, gated=0, split=0, acc=0):
